@@ -199,7 +199,7 @@ template <int BN, int kAct = ACT_NONE>
 __global__ void __launch_bounds__(GEMM_THREADS, 1)
     gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmap_a,
                      const __grid_constant__ CUtensorMap tmap_b, bf16* __restrict__ C, int M,
-                     int N, int K, int dbg, int splits, float* __restrict__ ws, int a_bytes) {
+                     int N, int K, int splits, float* __restrict__ ws, int a_bytes) {
   constexpr bool kSwiGLU = kAct != ACT_NONE;
   // a_bytes: bytes one A k-block really carries.  For M < 128 the tensor map's box holds only the
   // rows that exist (rounded up to the 8-row swizzle atom), not 128: the other rows of the UMMA's A
@@ -261,13 +261,9 @@ __global__ void __launch_bounds__(GEMM_THREADS, 1)
           mbar_wait(empty + stage, phase ^ 1u);
           uint8_t* sa = smem + stage * Cfg::STAGE_BYTES;
           uint8_t* sb = sa + Cfg::A_BYTES;
-          if (dbg & 1) {  // timing experiment: MMA on stale smem, no operand traffic
-            mbar_arrive(full + stage);
-          } else {
-            mbar_expect_tx(full + stage, (uint32_t)(a_bytes + Cfg::B_BYTES));
-            tma_load_2d(sa, &tmap_a, (kb0 + kb) * GEMM_BK, m_blk * GEMM_BM, full + stage);
-            tma_load_2d(sb, &tmap_b, (kb0 + kb) * GEMM_BK, n_blk * BN, full + stage);
-          }
+          mbar_expect_tx(full + stage, (uint32_t)(a_bytes + Cfg::B_BYTES));
+          tma_load_2d(sa, &tmap_a, (kb0 + kb) * GEMM_BK, m_blk * GEMM_BM, full + stage);
+          tma_load_2d(sb, &tmap_b, (kb0 + kb) * GEMM_BK, n_blk * BN, full + stage);
           if (++stage == STAGES) {
             stage = 0;
             phase ^= 1u;
@@ -340,7 +336,7 @@ __global__ void __launch_bounds__(GEMM_THREADS, 1)
               st_v4(wrow + c0 + 4 * j, make_uint4(v[4 * j], v[4 * j + 1], v[4 * j + 2], v[4 * j + 3]));
           }
         }
-      } else if (!(dbg & 2)) {  // dbg&2: skip the drain (timing experiment)
+      } else {
         epilogue_rows<BN, kAct>(taddr, ctile, ldc, row0, M, epi_smem + (warp - 2) * EPI_SMEM_PER_WARP, lane);
       }
       tc_fence_before();
@@ -470,7 +466,7 @@ template <int BN, int kAct = ACT_NONE>
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(GEMM_THREADS, 1)
     gemm2_bf16_kernel(const __grid_constant__ CUtensorMap tmap_a,
                       const __grid_constant__ CUtensorMap tmap_b, bf16* __restrict__ C, int M,
-                      int N, int K, int dbg) {
+                      int N, int K) {
   constexpr bool kSwiGLU = kAct != ACT_NONE;
   using Cfg = Gemm2Cfg<BN>;
   constexpr int STAGES = Cfg::STAGES;
@@ -526,13 +522,9 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(GEMM_THREADS, 1)
           uint8_t* sa = smem + stage * Cfg::STAGE_BYTES;
           uint8_t* sb = sa + Cfg::A_BYTES;
           const uint32_t lfull = mapa_shared(full + stage, 0);
-          if (dbg & 1) {  // timing experiment: MMA on stale smem, no operand traffic
-            mbar_arrive_cluster(lfull);
-          } else {
-            mbar_expect_tx_cluster(lfull, Cfg::STAGE_BYTES);
-            tma_load_2d_2sm(sa, &tmap_a, kb * GEMM_BK, m_blk * 256 + (int)rank * 128, lfull);
-            tma_load_2d_2sm(sb, &tmap_b, kb * GEMM_BK, n_blk * BN + (int)rank * (BN / 2), lfull);
-          }
+          mbar_expect_tx_cluster(lfull, Cfg::STAGE_BYTES);
+          tma_load_2d_2sm(sa, &tmap_a, kb * GEMM_BK, m_blk * 256 + (int)rank * 128, lfull);
+          tma_load_2d_2sm(sb, &tmap_b, kb * GEMM_BK, n_blk * BN + (int)rank * (BN / 2), lfull);
           if (++stage == STAGES) {
             stage = 0;
             phase ^= 1u;
@@ -590,8 +582,7 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(GEMM_THREADS, 1)
       const long long ldc = kSwiGLU ? N / 2 : N;
       bf16* ctile = C + (long long)row0 * ldc + (long long)n_blk * OUT_BN;
       const uint32_t taddr = tmem_base + ((uint32_t)(quarter * 32) << 16) + (uint32_t)(acc * BN);
-      if (!(dbg & 2))  // dbg&2: skip the drain (timing experiment)
-        epilogue_rows<BN, kAct>(taddr, ctile, ldc, row0, M, epi_smem + (warp - 2) * EPI_SMEM_PER_WARP, lane);
+      epilogue_rows<BN, kAct>(taddr, ctile, ldc, row0, M, epi_smem + (warp - 2) * EPI_SMEM_PER_WARP, lane);
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive_cluster(mapa_shared(tmem_empty + acc, 0));
@@ -702,8 +693,6 @@ static int num_sms() {
   return n;
 }
 
-static int g_gemm_debug = 0;  // timing experiments only (wrong results): 1 = no TMA loads, 2 = no epilogue
-
 static float* g_splitk_ws = nullptr;
 static size_t g_splitk_ws_bytes = 0;
 
@@ -739,7 +728,7 @@ static int launch_gemm(const void* A, const void* W, void* C, int M, int N, int 
     }
     ws = g_splitk_ws;
   }
-  kern<<<grid, GEMM_THREADS, Cfg::SMEM_TOTAL, st>>>(ta, tb, (bf16*)C, M, N, K, g_gemm_debug, splits, ws,
+  kern<<<grid, GEMM_THREADS, Cfg::SMEM_TOTAL, st>>>(ta, tb, (bf16*)C, M, N, K, splits, ws,
                                                     a_rows * GEMM_BK * 2);
   B200Q_LAUNCH_CHECK();
   if (partials_out) *partials_out = ws;  // the caller fuses the reduction into the consumer of C
@@ -795,7 +784,7 @@ static int launch_gemm2(const void* A, const void* W, void* C, int M, int N, int
     g_gemm2_pairs = pairs;
   }
   const int grid = 2 * (tiles < pairs ? tiles : pairs);
-  kern<<<grid, GEMM_THREADS, Cfg::SMEM_TOTAL, st>>>(ta, tb, (bf16*)C, M, N, K, g_gemm_debug);
+  kern<<<grid, GEMM_THREADS, Cfg::SMEM_TOTAL, st>>>(ta, tb, (bf16*)C, M, N, K);
   B200Q_LAUNCH_CHECK();
   return B200Q_OK;
 }
@@ -1190,13 +1179,6 @@ int b200q_gemm_set_tile_n(int bn) {
 // test/tuning hook: 0 = auto, 1 = 1-CTA kernels only, 2 = 2-CTA (cta_group::2) kernel whenever legal
 // diagnostics: co-resident CTA pairs the 2-CTA kernel's grid is sized to (0 until first use)
 int b200q_gemm_resident_pairs(void) { return g_gemm2_pairs; }
-
-// timing experiments only — results are garbage: bit0 skips the operand loads, bit1 the epilogue
-int b200q_gemm_set_debug(int flags) {
-  g_gemm_debug = flags & 3;
-  bump_tuning_epoch();
-  return B200Q_OK;
-}
 
 // test/tuning hook: 0 = auto split-K, 1 = off, n > 1 = force n splits (decode-sized M only)
 int b200q_gemm_set_splitk(int n) {
