@@ -30,7 +30,7 @@
 extern "C" {
 #endif
 
-#define B200Q_VERSION 5
+#define B200Q_VERSION 6
 
 #define B200Q_OK 0
 #define B200Q_EINVAL (-1)   /* bad argument / unsupported shape            */
@@ -516,6 +516,51 @@ int b200q_latent_attn_ex(const float* qa_dev, const void* cache_dev, const int32
                          int rot_dim, int block_size, int window, float scale, const void* gate_dev, int ld_gate,
                          void* out_dev, int dtype, void* stream);
 
+/* ---- parallel layers with one shared norm, differential attention (parallel_ops.cu, diff_attn.cu) ---------------- */
+
+/* x[t] += y[t] + bias (fp32 [W] or NULL), then out[t] = x / sqrt(mean(x^2) + eps) * (1 + w) in the model dtype (out
+ * NULL: the sum only).  y: model-dtype rows, or with y_f32 the sum over `splits` of fp32 [splits][T][W] in order (what
+ * b200q_gemm_bf16_splitk leaves) */
+int b200q_layer_close(float* x_dev, const void* y_dev, int y_f32, int splits, const float* bias_dev, const float* w_dev,
+                      void* out_dev, int T, int W, float eps, int dtype, void* stream);
+/* b200q_clamped_glu over rows of stride ld_in / ld_out with biases (fp32, indexed like a row; NULL: none) and gate / up
+ * columns side by side (block 0) or interleaved in blocks of `block` columns (block must divide F) */
+int b200q_clamped_glu_ex(const void* gate_up_dev, int ld_in, const float* bias_dev, void* y_dev, int ld_out, int64_t rows,
+                         int F, int block, float limit, int dtype, void* stream);
+/* fused gate_up GEMM + clamped unit: C[M, N/2] (rows of ldc elements); weight rows and bias (fp32 [N]) interleaved in
+ * blocks of 128 as for b200q_gemm_swiglu_bf16; the unit works on the fp32 accumulators */
+int b200q_gemm_clamped_glu_bf16(const void* A_dev, const void* W_dev, const float* bias_dev, void* C_dev, int ldc, int M,
+                                int N, int K, float limit, void* stream);
+/* table[t][i] = (cos, sin)(positions[t] * freq[i]) * mag, fp32 pairs [T][half], i < half; angles and functions in fp64 */
+int b200q_rot_table(const double* freq_dev, float mag, const int32_t* positions_dev, int T, int half, float* table_dev,
+                    void* stream);
+/* 1 if differential attention of these sizes runs on the tensor cores (bf16, pages of 16 rows, dim and vdim multiples
+ * of 16 up to 128, 2*dim + vdim a multiple of 64): queries are then bf16 with scale * log2 e folded in and cache rows are
+ * permuted; otherwise queries are fp32 with the scale folded in and cache rows lie as they are */
+int b200q_diff_attn_tiled(int dim, int vdim, int block_size, int dtype);
+/* differential attention 1/2: proj rows [q (heads*2*dim) | k (kv_heads*2*dim) | v (kv_heads*vdim) | ...] (own 0: [q |
+ * ...], the layer reads another layer's cache), each head's q and k as [map 1 | map 2].  Every channel: + bias (fp32,
+ * indexed like a row; NULL: none); y_t = sum_j conv[j][c] u_(t - taps + 1 + j) (conv: fp32 [taps][channels], taps 0: off;
+ * zeros before the sequence's start; the last taps - 1 values u travel in `state`, fp32 [taps - 1][channels]); of q and k
+ * the pairs (2i, 2i + 1) of a map's first rot_dims dimensions are turned by `table` (b200q_rot_table).  q: [T, heads, 2,
+ * dim] as b200q_diff_attn_tiled says; cache: [block][kv_heads][block_size][2*dim + vdim] = [key 1 | key 2 | value]. */
+int b200q_diff_attn_prep(const void* proj_dev, int ldp, const float* bias_dev, const float* conv_dev, int taps,
+                         float* state_dev, long long slot_stride, int own, int heads, int kv_heads, int dim, int vdim,
+                         int rot_dims, const float* table_dev, float scale, const int32_t* seq_desc_dev,
+                         const int32_t* row_seq_dev, int n_seqs, const int32_t* slot_mapping_dev, int block_size,
+                         void* q_dev, void* cache_dev, int T, int dtype, void* stream);
+/* differential attention 2/2: with a1, a2 the softmax attentions of a head's two maps over the keys j <= p of the token's
+ * sequence, o = a1 - lambda a2 (lambda: one fp32 number), out[t, h*vdim ..] = o / sqrt(mean(o^2) + eps) * mult *
+ * sigmoid(gate[t, h]) (gate NULL: 1); out rows of ld_out elements, gate rows of ld_gate */
+int b200q_diff_attn(const void* q_dev, const void* cache_dev, const int32_t* block_table_dev, int bt_stride,
+                    const int32_t* row_seq_dev, const int32_t* positions_dev, const int32_t* seq_desc_dev, int n_seqs,
+                    int T, int heads, int kv_heads, int dim, int vdim, int block_size, const float* lambda_dev,
+                    float mult, float eps, const void* gate_dev, int ld_gate, void* out_dev, int ld_out, int dtype,
+                    void* stream);
+/* nonzero once a kernel's bounded wait has run out in this process (its outputs are then missing); engine steps report
+ * it as B200Q_ECUDA */
+int b200q_wait_failures(void);
+
 /* ------------------------------------------------------------------------------------
  * Model-level: one forward step over a mixed decode+prefill token batch.
  * Replaces GPUModelRunner.execute_model for LlamaForCausalLM
@@ -564,6 +609,8 @@ typedef struct b200q_model_config {
   float residual_mult;    /* every sublayer's normed output is multiplied by this before it joins x; 0 = 1      */
   int32_t side_dim;       /* per-layer token input: columns of the second embedding table a layer reads; 0 = none */
   float logit_scale;      /* layered architectures: logits are multiplied by this; 0 = 1                        */
+  int32_t shared_norm;    /* parallel form, 1: both sublayers of a layer read norm1's output; the layer's projections
+                             are fused ("in", "in_b", "out", "out_b", see b200q_model_create_layered)             */
 } b200q_model_config;
 
 #define B200Q_ARCH_LLAMA 0
@@ -591,6 +638,13 @@ typedef struct b200q_model_config {
  * logarithm of the position, keys and values shared with an earlier layer; latent attention with full-rank queries,
  * YaRN-scaled frequencies and a sigmoid gate per head; gated GELU feed-forwards; scaled logits. */
 #define B200Q_ARCH_KABAVIK 5
+
+/* Lipedra: a layered decoder in parallel form with ONE norm per layer, read by both sublayers,
+ *   h = norm1 x;  x <- x + mixer(h) + ff(h)
+ * (zero-centred RMS norms); differential attention (two softmax maps per head over the same values, subtracted and
+ * normed) with biases, short convolutions on q, k and v, interleaved rotation with YaRN frequencies, a gate number per
+ * head and optionally an earlier layer's keys and values; a clamped gated feed-forward with biases. */
+#define B200Q_ARCH_LIPEDRA 6
 
 #define B200Q_FORM_PARALLEL 0  /* x <- x + mixer(norm1 x) + ff(norm2 x)                                  */
 #define B200Q_FORM_POSTNORM 1  /* x <- norm1(alpha x + ls1 mixer(x~)); x <- norm2(alpha x + ls2 ff(x~)) */
@@ -627,6 +681,10 @@ typedef struct b200q_model_config {
  * the input with the previous token's input; w = exp(-exp(w0 + W2 tanh(W1 .))); o = (S + diag(u) k v^T)^T r,
  * S <- diag(w) S + k v^T; per-head RMS, a weight, a SiLU gate                                                  */
 #define B200Q_MIXER_DECAY_MIX 8
+/* differential attention: per head two query / key maps of `dim` over shared values of `vdim`, o = a1 - lambda a2,
+ * o / rms(o) * (1 - diff) * sigmoid(gate number of the head); q, k, v have biases and pass a causal convolution of
+ * conv_taps taps per channel before the leading rot_dims of every map are turned (pairs 2i, 2i+1)             */
+#define B200Q_MIXER_DIFF_ATTN 9
 #define B200Q_FF_NONE 0
 #define B200Q_FF_POLYNORM 1         /* down(PolyNorm(up h))                                                          */
 #define B200Q_FF_MOE 2              /* top-k of clamped gated experts + an optional gated shared expert              */
@@ -641,6 +699,9 @@ typedef struct b200q_model_config {
 #define B200Q_FF_GEGLU 6            /* down(gelu_tanh(gate h) * up h); "mlp.gate_up" [2*ff, W] = gate rows, then up rows,
                                        or "mlp.gate_up_il" = the same rows interleaved in blocks of 128 (ff a multiple
                                        of 128), which a bf16 model runs with the unit in the product's epilogue */
+
+#define B200Q_FF_CLAMPED 7          /* down(g' sigmoid(1.702 g') (u' + 1)), g' = min(gate h, ff_limit), u' = clamp(up h,
+                                       -ff_limit, ff_limit); all three projections have biases (shared-norm layers)  */
 
 typedef struct b200q_layer_desc {
   int32_t mixer;        /* B200Q_MIXER_*                                                               */
@@ -702,6 +763,9 @@ typedef struct b200q_layer_desc {
    * dim(rot_fast)), 0), hi = min(ceil(dim(rot_slow)), rot_dims - 1), r_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1):
    * f_i / rot_factor * r_i + f_i (1 - r_i), and sine and cosine are multiplied by 0.1 ln(rot_factor) + 1 */
   double rot_factor, rot_original, rot_fast, rot_slow;
+  /* differential attention and the clamped feed-forward (zero elsewhere) */
+  float diff;           /* differential attention: heads' outputs are multiplied by 1 - diff               */
+  float ff_limit;       /* clamped feed-forward                                                            */
 } b200q_layer_desc;
 
 typedef struct b200q_model* b200q_model_t;
@@ -768,7 +832,13 @@ int b200q_model_create(const b200q_model_config* cfg, b200q_model_t* out);
  *   selective scan: "mix.proj" [2*inner, W] (rows: x, z), "mix.conv" [1, inner*conv_taps], "mix.conv_b" [1, inner],
  *     "mix.x" [roundup64(dt_rank + 2*state_dim), inner] (rows: dt, B, C, then zero rows), "mix.dt" [inner, dt_rank],
  *     "mix.dt_b" [1, inner], "mix.a_log" [1, inner*state_dim], "mix.d" [1, inner], "mix.o" [W, inner]
- *   sigmoid-routed experts: "mlp.router" [E, W], "mlp.experts_gate_up" [E*2*ff, W], "mlp.experts_down" [E*W, ff] */
+ *   sigmoid-routed experts: "mlp.router" [E, W], "mlp.experts_gate_up" [E*2*ff, W], "mlp.experts_down" [E*W, ff]
+ * B200Q_ARCH_LIPEDRA (cfg.layer_form = B200Q_FORM_PARALLEL, cfg.shared_norm = 1): per layer "norm1" [1, W], "mix.conv"
+ *   [1, conv_taps*channels] ([taps][channels of q | k | v]; with conv_taps > 0), "mix.lambda" [1, 1], and the fused
+ *   projections: "in" [NP + 2*ff, W] = rows q | k | v (own keys and values) | gate numbers | zero rows up to NP, then
+ *   gate | up rows of the feed-forward ("in_il": interleaved in blocks of 128, ff a multiple of 128); "in_b" [1, NP +
+ *   2*ff] their biases in the same order; "out" [W, heads*vdim + ff] = [output projection | down projection]; "out_b"
+ *   [1, W] (with a feed-forward).  NP is a multiple of 256 from 1024 used rows up, else of 64. */
 int b200q_model_create_layered(const b200q_model_config* cfg, const b200q_layer_desc* layers,
                                b200q_model_t* out);
 /* layered models: bytes of one cache block over all layers that own a latent cache (the caller allocates

@@ -430,6 +430,10 @@ static int complete_step(b200q_engine* e, InFlightStep& st, int64_t* out_req_ids
       set_error("step: forward failed: %s", cudaGetErrorString(ce));
       return B200Q_ECUDA;
     }
+    if (b200q_wait_failures()) {
+      set_error("step: a kernel's bounded wait ran out");
+      return B200Q_ECUDA;
+    }
   }
   const int32_t* h_out = e->h_out_buf[st.buf];
   int n_ev = *n_out;
@@ -972,6 +976,10 @@ int b200q_engine_step_replay(b200q_engine_t e, int32_t n_entries, const int64_t*
   if (!rc) rc = launch_step(e, st, sched, logits_out);
   if (!rc && !e->dry_run && cudaStreamSynchronize(e->stream) != cudaSuccess) {
     set_error("step_replay: forward failed: %s", cudaGetErrorString(cudaGetLastError()));
+    rc = B200Q_ECUDA;
+  }
+  if (!rc && b200q_wait_failures()) {
+    set_error("step_replay: a kernel's bounded wait ran out");
     rc = B200Q_ECUDA;
   }
   for (StepEntry& se : st.entries) se.r->refs--;

@@ -2,7 +2,7 @@
 // for the QKV / O / gate_up / down / LM-head projections (SURVEY.md §2.1 K3,K8,K9,K11,K12),
 // the only dense contractions of the hot path.  Hand-written for sm_100a:
 //
-//   * persistent, warp-specialised CTA (192 threads): warp 0 = TMA producer (UTMALDG, 128B
+//   * persistent, warp-specialised CTA (192 threads): warp 0 = TMA producer (128B
 //     swizzle), warp 1 = tcgen05.mma issuer (one lane; also owns the TMEM allocation),
 //     warps 2-5 = epilogue (tcgen05.ld -> bf16 -> global).
 //   * tile 128 x BN x 64 (BN in {64,128,256}), smem ring of 4..8 stages (<= 192 KB), operands
@@ -126,11 +126,18 @@ constexpr int EPI_SMEM_PER_WARP = 32 * 128;  // 32 rows x 64 bf16
 // kAct: 0 = plain GEMM, 1 = SwiGLU (Llama), 2 = GeGLU with the tanh approximation (Gemma-2):
 // out = bf16(bf16(gelu_tanh(bf16(g))) * bf16(u)), gelu_tanh evaluated in fp32 like torch's kernel:
 // 0.5 * g * (1 + tanh(sqrt(2/pi) * (g + 0.044715 g^3)))
-constexpr int ACT_NONE = 0, ACT_SWIGLU = 1, ACT_GEGLU = 2;
+// 3 = clamped unit with biases (Lipedra): g' sigmoid(1.702 g') (u' + 1), g' = min(g + bg, limit), u' = clamp(u + bu,
+// -limit, limit), in fp32 from the accumulators (one rounding); bias: fp32, this tile's [gate (BN/2) | up (BN/2)]
+constexpr int ACT_NONE = 0, ACT_SWIGLU = 1, ACT_GEGLU = 2, ACT_CLAMPED = 3;
+struct GateArgs {
+  const float* bias;
+  float limit;
+};
 
 template <int BN, int kAct>
 __device__ __forceinline__ void epilogue_rows(uint32_t taddr, bf16* ctile, long long ldc,
-                                              int row0, int M, uint8_t* patch, int lane) {
+                                              int row0, int M, uint8_t* patch, int lane,
+                                              const float* gate_bias = nullptr, float limit = 0.f) {
   constexpr bool kSwiGLU = kAct != ACT_NONE;  // gated epilogue: tile = [gate (BN/2) | up (BN/2)]
   constexpr int OUT_BN = kSwiGLU ? BN / 2 : BN;
   auto act = [](uint32_t gb, uint32_t ub) -> float {
@@ -164,6 +171,30 @@ __device__ __forceinline__ void epilogue_rows(uint32_t taddr, bf16* ctile, long 
         tmem_ld32(taddr + (uint32_t)(c0 + 32 * h), v);
         tmem_ld32(taddr + (uint32_t)(BN / 2 + c0 + 32 * h), u);
         tmem_ld_wait();
+        if constexpr (kAct == ACT_CLAMPED) {
+          const float4* bg = reinterpret_cast<const float4*>(gate_bias + c0 + 32 * h);
+          const float4* bu = reinterpret_cast<const float4*>(gate_bias + BN / 2 + c0 + 32 * h);
+          auto unit = [&](uint32_t gb, uint32_t ub, float b0, float b1) -> uint32_t {
+            const float g = fminf(__uint_as_float(gb) + b0, limit);
+            const float w = fminf(fmaxf(__uint_as_float(ub) + b1, -limit), limit);
+            return __float_as_uint(g / (1.f + __expf(-1.702f * g)) * (w + 1.f));
+          };
+#pragma unroll
+          for (int j = 0; j < 8; ++j) {
+            const float4 x = __ldg(bg + j), y = __ldg(bu + j);
+            v[4 * j + 0] = unit(v[4 * j + 0], u[4 * j + 0], x.x, y.x);
+            v[4 * j + 1] = unit(v[4 * j + 1], u[4 * j + 1], x.y, y.y);
+            v[4 * j + 2] = unit(v[4 * j + 2], u[4 * j + 2], x.z, y.z);
+            v[4 * j + 3] = unit(v[4 * j + 3], u[4 * j + 3], x.w, y.w);
+          }
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            o[j].x = pack_bf16x2(__uint_as_float(v[8 * j + 0]), __uint_as_float(v[8 * j + 1]));
+            o[j].y = pack_bf16x2(__uint_as_float(v[8 * j + 2]), __uint_as_float(v[8 * j + 3]));
+            o[j].z = pack_bf16x2(__uint_as_float(v[8 * j + 4]), __uint_as_float(v[8 * j + 5]));
+            o[j].w = pack_bf16x2(__uint_as_float(v[8 * j + 6]), __uint_as_float(v[8 * j + 7]));
+          }
+        } else
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           o[j].x = pack_bf16x2(act(v[8 * j + 0], u[8 * j + 0]), act(v[8 * j + 1], u[8 * j + 1]));
@@ -199,7 +230,8 @@ template <int BN, int kAct = ACT_NONE>
 __global__ void __launch_bounds__(GEMM_THREADS, 1)
     gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmap_a,
                      const __grid_constant__ CUtensorMap tmap_b, bf16* __restrict__ C, int M,
-                     int N, int K, int splits, float* __restrict__ ws, int a_bytes) {
+                     int N, int K, int splits, float* __restrict__ ws, int a_bytes,
+                     long long ldc, GateArgs gate) {
   constexpr bool kSwiGLU = kAct != ACT_NONE;
   // a_bytes: bytes one A k-block really carries.  For M < 128 the tensor map's box holds only the
   // rows that exist (rounded up to the 8-row swizzle atom), not 128: the other rows of the UMMA's A
@@ -318,7 +350,6 @@ __global__ void __launch_bounds__(GEMM_THREADS, 1)
       tc_fence_after();
       const int row0 = m_blk * GEMM_BM + quarter * 32;
       constexpr int OUT_BN = kSwiGLU ? BN / 2 : BN;
-      const long long ldc = kSwiGLU ? N / 2 : N;
       bf16* ctile = C + (long long)row0 * ldc + (long long)n_blk * OUT_BN;
       const uint32_t taddr = tmem_base + ((uint32_t)(quarter * 32) << 16) + (uint32_t)(acc * BN);
       if (splits > 1) {
@@ -337,7 +368,8 @@ __global__ void __launch_bounds__(GEMM_THREADS, 1)
           }
         }
       } else {
-        epilogue_rows<BN, kAct>(taddr, ctile, ldc, row0, M, epi_smem + (warp - 2) * EPI_SMEM_PER_WARP, lane);
+        epilogue_rows<BN, kAct>(taddr, ctile, ldc, row0, M, epi_smem + (warp - 2) * EPI_SMEM_PER_WARP, lane,
+                                kAct == ACT_CLAMPED ? gate.bias + (long long)n_blk * BN : nullptr, gate.limit);
       }
       tc_fence_before();
       __syncwarp();
@@ -466,7 +498,7 @@ template <int BN, int kAct = ACT_NONE>
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(GEMM_THREADS, 1)
     gemm2_bf16_kernel(const __grid_constant__ CUtensorMap tmap_a,
                       const __grid_constant__ CUtensorMap tmap_b, bf16* __restrict__ C, int M,
-                      int N, int K) {
+                      int N, int K, long long ldc, GateArgs gate) {
   constexpr bool kSwiGLU = kAct != ACT_NONE;
   using Cfg = Gemm2Cfg<BN>;
   constexpr int STAGES = Cfg::STAGES;
@@ -579,10 +611,10 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(GEMM_THREADS, 1)
       tc_fence_after();
       const int row0 = m_blk * 256 + (int)rank * 128 + quarter * 32;
       constexpr int OUT_BN = kSwiGLU ? BN / 2 : BN;
-      const long long ldc = kSwiGLU ? N / 2 : N;
       bf16* ctile = C + (long long)row0 * ldc + (long long)n_blk * OUT_BN;
       const uint32_t taddr = tmem_base + ((uint32_t)(quarter * 32) << 16) + (uint32_t)(acc * BN);
-      epilogue_rows<BN, kAct>(taddr, ctile, ldc, row0, M, epi_smem + (warp - 2) * EPI_SMEM_PER_WARP, lane);
+      epilogue_rows<BN, kAct>(taddr, ctile, ldc, row0, M, epi_smem + (warp - 2) * EPI_SMEM_PER_WARP, lane,
+                                kAct == ACT_CLAMPED ? gate.bias + (long long)n_blk * BN : nullptr, gate.limit);
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive_cluster(mapa_shared(tmem_empty + acc, 0));
@@ -698,7 +730,8 @@ static size_t g_splitk_ws_bytes = 0;
 
 template <int BN, int kAct = ACT_NONE>
 static int launch_gemm(const void* A, const void* W, void* C, int M, int N, int K,
-                       cudaStream_t st, int splits = 1, const float** partials_out = nullptr) {
+                       cudaStream_t st, int splits = 1, const float** partials_out = nullptr, long long ldc = 0,
+                       GateArgs gate = {nullptr, 0.f}) {
   using Cfg = GemmCfg<BN>;
   CUtensorMap ta, tb;
   const int a_rows = M < GEMM_BM ? (M + 7) & ~7 : GEMM_BM;  // one m-tile: load only the rows that exist
@@ -729,7 +762,8 @@ static int launch_gemm(const void* A, const void* W, void* C, int M, int N, int 
     ws = g_splitk_ws;
   }
   kern<<<grid, GEMM_THREADS, Cfg::SMEM_TOTAL, st>>>(ta, tb, (bf16*)C, M, N, K, splits, ws,
-                                                    a_rows * GEMM_BK * 2);
+                                                    a_rows * GEMM_BK * 2,
+                                                    ldc > 0 ? ldc : (kAct != ACT_NONE ? N / 2 : N), gate);
   B200Q_LAUNCH_CHECK();
   if (partials_out) *partials_out = ws;  // the caller fuses the reduction into the consumer of C
   if (splits > 1 && !partials_out) {
@@ -745,7 +779,7 @@ static int g_gemm2_pairs = 0;  // co-resident CTA pairs reported by the occupanc
 
 template <int BN, int kAct = ACT_NONE>
 static int launch_gemm2(const void* A, const void* W, void* C, int M, int N, int K,
-                        cudaStream_t st) {
+                        cudaStream_t st, long long ldc = 0, GateArgs gate = {nullptr, 0.f}) {
   using Cfg = Gemm2Cfg<BN>;
   CUtensorMap ta, tb;
   int rc = get_tmap(A, M, K, GEMM_BM, &ta);
@@ -784,7 +818,8 @@ static int launch_gemm2(const void* A, const void* W, void* C, int M, int N, int
     g_gemm2_pairs = pairs;
   }
   const int grid = 2 * (tiles < pairs ? tiles : pairs);
-  kern<<<grid, GEMM_THREADS, Cfg::SMEM_TOTAL, st>>>(ta, tb, (bf16*)C, M, N, K);
+  kern<<<grid, GEMM_THREADS, Cfg::SMEM_TOTAL, st>>>(ta, tb, (bf16*)C, M, N, K,
+                                                  ldc > 0 ? ldc : (kAct != ACT_NONE ? N / 2 : N), gate);
   B200Q_LAUNCH_CHECK();
   return B200Q_OK;
 }
@@ -1091,7 +1126,7 @@ using namespace b200q;
 // shared body of the fused gate_up GEMMs (SwiGLU / GeGLU)
 template <int kAct>
 static int gemm_gated(const char* what, const void* A, const void* W, void* C, int M, int N, int K,
-                      void* stream) {
+                      void* stream, long long ldc = 0, GateArgs gate = {nullptr, 0.f}) {
   B200Q_CHECK_ARG(M >= 0 && N > 0 && K > 0 && K % GEMM_BK == 0 && N % 256 == 0,
                   "%s: unsupported shape M=%d N=%d K=%d (need K%%64==0, N%%256==0)", what, M, N, K);
   B200Q_CHECK_ARG((reinterpret_cast<uintptr_t>(A) & 15) == 0 &&
@@ -1101,8 +1136,8 @@ static int gemm_gated(const char* what, const void* A, const void* W, void* C, i
   if (M == 0) return B200Q_OK;
   cudaStream_t st = as_stream(stream);
   if ((g_gemm_mode == 2 && M > GEMM_BM) || (g_gemm_mode == 0 && prefer_2cta(M, N)))
-    return launch_gemm2<256, kAct>(A, W, C, M, N, K, st);
-  return launch_gemm<256, kAct>(A, W, C, M, N, K, st);
+    return launch_gemm2<256, kAct>(A, W, C, M, N, K, st, ldc, gate);
+  return launch_gemm<256, kAct>(A, W, C, M, N, K, st, 1, nullptr, ldc, gate);
 }
 
 extern "C" {
@@ -1282,6 +1317,14 @@ int b200q_gemm_swiglu_bf16(const void* A, const void* W, void* C, int M, int N, 
 // Gemma-2's GeGLU (gelu_tanh(gate) * up) in the same fused epilogue, same weight interleaving
 int b200q_gemm_geglu_bf16(const void* A, const void* W, void* C, int M, int N, int K, void* stream) {
   return gemm_gated<ACT_GEGLU>("gemm_geglu", A, W, C, M, N, K, stream);
+}
+
+// the clamped gated unit with biases in the same epilogue; C has rows of ldc elements
+int b200q_gemm_clamped_glu_bf16(const void* A, const void* W, const float* bias, void* C, int ldc, int M, int N, int K,
+                                float limit, void* stream) {
+  B200Q_CHECK_ARG(bias && ldc >= N / 2 && ldc % 8 == 0 && (reinterpret_cast<uintptr_t>(bias) & 15) == 0 && limit >= 0.f,
+                  "gemm_clamped_glu: bad bias, row stride (%d) or limit", ldc);
+  return gemm_gated<ACT_CLAMPED>("gemm_clamped_glu", A, W, C, M, N, K, stream, ldc, GateArgs{bias, limit});
 }
 
 }  // extern "C"

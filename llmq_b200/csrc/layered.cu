@@ -61,7 +61,7 @@ int check_sequence_mixer(int i, const b200q_layer_desc& d) {
 int check_layered(const b200q_model_config* c, const b200q_layer_desc* L) {
   B200Q_CHECK_ARG(c && L, "layered config is null");
   B200Q_CHECK_ARG(c->arch == B200Q_ARCH_RAMOPEL || c->arch == B200Q_ARCH_NORIDRA || c->arch == B200Q_ARCH_PALUZEN ||
-                      c->arch == B200Q_ARCH_KABAVIK,
+                      c->arch == B200Q_ARCH_KABAVIK || c->arch == B200Q_ARCH_LIPEDRA,
                   "create_layered: arch=%d is not a layered architecture", c->arch);
   B200Q_CHECK_ARG(c->layer_form == B200Q_FORM_PARALLEL || c->layer_form == B200Q_FORM_POSTNORM ||
                       c->layer_form == B200Q_FORM_PRENORM || c->layer_form == B200Q_FORM_SANDWICH,
@@ -72,6 +72,8 @@ int check_layered(const b200q_model_config* c, const b200q_layer_desc* L) {
                            : (c->norm_kind == 0 && c->side_dim == 0 && c->residual_mult == 0.f),
                   "norm kind (%d), residual multiplier and per-layer token input belong to the sandwich form",
                   c->norm_kind);
+  B200Q_CHECK_ARG(c->shared_norm == 0 || (c->shared_norm == 1 && c->layer_form == B200Q_FORM_PARALLEL && c->learned_pos == 0),
+                  "a norm shared by both sublayers belongs to the parallel form");
   B200Q_CHECK_ARG(c->logit_softcap >= 0.f && (c->token_shift == 0 || c->layer_form == B200Q_FORM_PRENORM),
                   "bad logit soft cap, or a token shift outside the pre-norm form");
   B200Q_CHECK_ARG(c->norm_groups >= 0 && (c->norm_groups <= 1 || c->hidden % c->norm_groups == 0) &&
@@ -124,6 +126,20 @@ int check_layered(const b200q_model_config* c, const b200q_layer_desc* L) {
                         "layer %d: kv_from=%d must name an earlier window-attention layer with keys and values of its "
                         "own and the same sizes", i, d.kv_from);
       }
+    } else if (d.mixer == B200Q_MIXER_DIFF_ATTN) {
+      B200Q_CHECK_ARG(d.heads > 0 && d.kv_heads > 0 && d.heads % d.kv_heads == 0 && d.dim > 0 && d.dim <= 256 && d.vdim > 0 &&
+                          d.vdim <= 512 && d.conv_taps >= 0 && d.conv_taps <= 16 && d.rot_dims >= 0 && d.rot_dims % 2 == 0 &&
+                          d.rot_dims <= d.dim && (d.rot_dims == 0 || d.rot_base > 0.0) && d.rot_factor >= 0.0 &&
+                          d.rot_original >= 0.0 && d.window == 0 && c->shared_norm,
+                      "layer %d: bad differential-attention sizes (dim <= 256, vdim <= 512, taps <= 16, even rot.dims <= dim, "
+                      "kv_heads divides heads; every earlier key; shared-norm layers)", i);
+      if (d.kv_from >= 0) {
+        const b200q_layer_desc& o = L[d.kv_from < i ? d.kv_from : 0];
+        B200Q_CHECK_ARG(d.kv_from < i && o.mixer == B200Q_MIXER_DIFF_ATTN && o.kv_from < 0 && o.kv_heads == d.kv_heads &&
+                            o.dim == d.dim && o.vdim == d.vdim,
+                        "layer %d: kv_from=%d must name an earlier differential-attention layer with keys and values of "
+                        "its own and the same sizes", i, d.kv_from);
+      }
     } else {
       set_error("layer %d: unknown mixer %d", i, d.mixer);
       return B200Q_EINVAL;
@@ -139,7 +155,11 @@ int check_layered(const b200q_model_config* c, const b200q_layer_desc* L) {
                     "layer %d: feed-forward %d is not built for the sandwich form", i, d.ff);
     B200Q_CHECK_ARG(!sandwich || d.mixer == B200Q_MIXER_LATENT_ATTN || d.mixer == B200Q_MIXER_WINDOW_ATTN,
                     "layer %d: mixer %d is not built for the sandwich form", i, d.mixer);
-    if (d.ff == B200Q_FF_GEGLU) {
+    B200Q_CHECK_ARG(!c->shared_norm || (d.mixer == B200Q_MIXER_DIFF_ATTN && (d.ff == B200Q_FF_CLAMPED || d.ff == B200Q_FF_NONE)),
+                    "layer %d: mixer %d / feed-forward %d are not built for layers with a shared norm", i, d.mixer, d.ff);
+    if (d.ff == B200Q_FF_CLAMPED) {
+      B200Q_CHECK_ARG(d.ff_dim > 0 && d.ff_limit >= 0.f && c->shared_norm, "layer %d: bad clamped feed-forward", i);
+    } else if (d.ff == B200Q_FF_GEGLU) {
       B200Q_CHECK_ARG(d.ff_dim > 0 && sandwich, "layer %d: bad gated-GELU feed-forward", i);
     } else if (d.ff == B200Q_FF_RELU2) {
       B200Q_CHECK_ARG(d.ff_dim > 0 && c->layer_form == B200Q_FORM_PRENORM, "layer %d: bad squared-ReLU feed-forward", i);
@@ -172,7 +192,7 @@ int check_layered(const b200q_model_config* c, const b200q_layer_desc* L) {
 // widest use of every workspace buffer over the layers
 struct Widths {
   int64_t proj = 1, cq = 1, q = 1, qa = 1, olat = 1, attn = 1, ffh = 1, ffa = 1, experts = 1, pairs = 1, egu = 1,
-          eact = 1, delta = 0, cvf = 0, baf = 0, dtr = 0, xc = 0, xp = 0, blend = 0;
+          eact = 1, delta = 0, cvf = 0, baf = 0, dtr = 0, xc = 0, xp = 0, blend = 0, rot = 0;
   bool moe = false, shared = false, hf = false, side = false, inject = false;
 };
 int64_t pad64(int64_t v) { return (v + 63) & ~(int64_t)63; }
@@ -187,6 +207,16 @@ int64_t window_proj_rows(const b200q_layer_desc& d) {
 int64_t latent_full_rows(const b200q_layer_desc& d) {
   return pad64((int64_t)d.heads * (d.dim + d.rot_dim) + d.kv_rank + d.rot_dim + d.heads);
 }
+// channels of differential attention's q | k | v (k and v with own keys), and the rows of its part of the fused input
+// projection: those channels, a gate number per head, zero rows
+int64_t diff_channels(const b200q_layer_desc& d) {
+  return (int64_t)d.heads * 2 * d.dim + (d.kv_from < 0 ? (int64_t)d.kv_heads * (2 * d.dim + d.vdim) : 0);
+}
+int64_t diff_proj_rows(const b200q_layer_desc& d) {
+  const int64_t n = diff_channels(d) + d.heads;
+  return n >= 1024 ? (n + 255) & ~(int64_t)255 : pad64(n);
+}
+int64_t clamped_ff(const b200q_layer_desc& d) { return d.ff == B200Q_FF_CLAMPED ? d.ff_dim : 0; }
 void sequence_mixer_widths(const b200q_layer_desc& d, int64_t W, Widths& w) {
   const int64_t HD = (int64_t)d.heads * d.dim, HV = (int64_t)d.heads * d.vdim;
   if (d.mixer == B200Q_MIXER_LIGHTNING) {
@@ -240,6 +270,11 @@ Widths widths_of(const b200q_model_config& c, const std::vector<b200q_layered_la
       w.xp = std::max<int64_t>(w.xp, (d.dt_rank + 2 * (int64_t)d.state_dim + 63) & ~(int64_t)63);
       w.dtr = std::max<int64_t>(w.dtr, d.inner);
       w.attn = std::max<int64_t>(w.attn, d.inner);
+    } else if (d.mixer == B200Q_MIXER_DIFF_ATTN) {
+      w.proj = std::max<int64_t>(w.proj, diff_proj_rows(d) + 2 * clamped_ff(d));
+      w.qa = std::max<int64_t>(w.qa, (int64_t)d.heads * 2 * d.dim);
+      w.attn = std::max<int64_t>(w.attn, (int64_t)d.heads * d.vdim + clamped_ff(d));
+      w.rot = std::max<int64_t>(w.rot, d.rot_dims);
     } else {
       sequence_mixer_widths(d, c.hidden, w);
     }
@@ -337,6 +372,7 @@ int64_t layout(b200q_model* m, uint8_t* base) {
   y->blend = take(w.blend ? T * w.blend * es : 1);
   y->tg = take(c.side_dim > 0 ? T * c.side_dim * es : 1);
   y->ta = take(c.side_dim > 0 ? T * c.side_dim * es : 1);
+  y->rot = (float*)take(w.rot ? T * w.rot * 4 : 1);
   y->sel = take(LR * W * es);
   y->logits = (float*)take(LR * (int64_t)c.vocab * 4);
   y->logits_bf16 = take((int64_t)c.max_seqs * c.vocab * 2);
@@ -411,6 +447,22 @@ int layered_create(const b200q_model_config* cfg, const b200q_layer_desc* layers
         m->lay->kv_block_bytes += (int64_t)cfg->block_size * l.d.kv_heads * (l.d.dim + l.d.vdim) * es;
       } else {  // the keys and values of an earlier layer, as its cache holds them
         l.cache_block_off = m->lay->layers[l.d.kv_from].cache_block_off;
+      }
+      if ((rc = upload_frequencies(l))) {
+        b200q_model_destroy(m);
+        return rc;
+      }
+    }
+    if (l.d.mixer == B200Q_MIXER_DIFF_ATTN) {
+      if (l.d.kv_from < 0) {
+        l.cache_block_off = m->lay->kv_block_bytes;
+        m->lay->kv_block_bytes += (int64_t)cfg->block_size * l.d.kv_heads * (2 * l.d.dim + l.d.vdim) * es;
+      } else {  // the keys and values of an earlier layer, as its cache holds them
+        l.cache_block_off = m->lay->layers[l.d.kv_from].cache_block_off;
+      }
+      if (l.d.conv_taps > 1) {
+        l.conv_off = m->lay->state_slot_floats;
+        m->lay->state_slot_floats += (int64_t)(l.d.conv_taps - 1) * diff_channels(l.d);
       }
       if ((rc = upload_frequencies(l))) {
         b200q_model_destroy(m);
@@ -534,6 +586,23 @@ int layered_bind_weight(b200q_model* m, const char* name, const void* p, int64_t
     }
   }
   FIELD("norm1", l.norm1, 1, W)
+  if (c.shared_norm) {
+    const int64_t NI = diff_proj_rows(d) + 2 * clamped_ff(d);
+    FIELD("in", l.in, NI, W)
+    if (!strcmp(field, "in_il")) {
+      B200Q_CHECK_ARG(clamped_ff(d) > 0 && d.ff_dim % 128 == 0,
+                      "layer %d: interleaved gate / up rows need ff (%d) to be a multiple of 128", li, d.ff_dim);
+      if ((rc = expect(NI, W))) return rc;
+      l.in = p;
+      l.gate_up_il = true;
+      return B200Q_OK;
+    }
+    FIELD("in_b", l.in_b, 1, NI)
+    FIELD("out", l.out, W, (int64_t)d.heads * d.vdim + clamped_ff(d))
+    if (clamped_ff(d) > 0) FIELD("out_b", l.out_b, 1, W)
+    if (d.conv_taps > 0) FIELD("mix.conv", l.conv_w, 1, d.conv_taps * diff_channels(d))
+    FIELD("mix.lambda", l.map_lambda, 1, 1)
+  }
   if (d.ff != B200Q_FF_NONE) FIELD("norm2", l.norm2, 1, W)
   if (c.token_shift) FIELD("shift", l.shift, 1, W)
   if (d.inject) FIELD("inject", l.inject, W, 2 * W)
@@ -689,7 +758,12 @@ static int check_bound(b200q_model* m) {
   for (size_t i = 0; i < m->lay->layers.size(); ++i) {
     const b200q_layered_layer& l = m->lay->layers[i];
     const b200q_layer_desc& d = l.d;
-    bool ok = l.norm1 && l.o && (d.ff == B200Q_FF_NONE || l.norm2);
+    bool ok = l.norm1 && (m->cfg.shared_norm || (l.o && (d.ff == B200Q_FF_NONE || l.norm2)));
+    if (m->cfg.shared_norm) {
+      need_kv = true;
+      if (d.conv_taps > 1) need_state = true;
+      ok = ok && l.in && l.in_b && l.out && l.map_lambda && (d.conv_taps == 0 || l.conv_w) && (clamped_ff(d) == 0 || l.out_b);
+    }
     if (m->cfg.layer_form == B200Q_FORM_POSTNORM) {
       ok = ok && l.ls1 && (d.ff == B200Q_FF_NONE || l.ls2);
       if (m->cfg.input_taps > 0) ok = ok && l.canon1 && (d.ff == B200Q_FF_NONE || l.canon2);
@@ -994,6 +1068,7 @@ int layered_forward(b200q_model* m, const b200q_batch* b, void* stream) {
   for (const auto& l : y->layers) keep_x0 = keep_x0 || l.d.inject;
   if (keep_x0) TRY(EW, 8.0 * T * W, b200q_copy_f32(y->x, y->x0, (int64_t)T * W, stream));
 
+  int rot_layer = -1;  // the layer whose rotation y->rot holds
   for (int li = 0; li < c.n_layers; ++li) {
     const b200q_layered_layer& l = y->layers[li];
     const b200q_layer_desc& d = l.d;
@@ -1105,6 +1180,61 @@ int layered_forward(b200q_model* m, const b200q_batch* b, void* stream) {
             b200q_sandwich_add(y->x, y->ffo, nullptr, B200Q_NORM_RMS, l.tok_norm, mult, next_kind, next_w, y->h1, T, W,
                                c.rms_eps, dt, stream));
       }
+      if (y->tap) TRY(EW, 8.0 * T * W, b200q_copy_f32(y->x, y->tap + (int64_t)li * T * W, (int64_t)T * W, stream));
+      continue;
+    }
+    if (c.shared_norm) {
+      // h = norm1 x;  x <- x + mixer(h) + ff(h): one product gives the rows of both sublayers, one product sums both
+      const int H = d.heads, G = d.kv_heads, HV = H * d.vdim, F = (int)clamped_ff(d), NP = (int)diff_proj_rows(d),
+                NI = NP + 2 * F, KO = HV + F, NC = (int)diff_channels(d);
+      const bool own = d.kv_from < 0;
+      if (li == 0)
+        TRY(EW, (double)T * W * (4 + es),
+            b200q_centered_rmsnorm(y->x, nullptr, l.norm1, nullptr, y->h1, nullptr, T, W, c.rms_eps, dt, stream));
+      uint8_t* act = (uint8_t*)y->attn + (size_t)HV * es;  // the unit's outputs lie behind the heads' in a row
+      // long steps of a bf16 model: the unit runs in the product's epilogue and the [T, 2F] activations are never written
+      // (shorter steps keep one product for both sublayers: its narrower tiles put more SMs on the weight stream)
+      const bool split = F > 0 && l.gate_up_il && dt == B200Q_DTYPE_BF16 && W % 64 == 0 && T >= 512 && HV % 8 == 0 &&
+                         KO % 8 == 0 && (reinterpret_cast<uintptr_t>(l.in) & 15) == 0;
+      const int ldp = split ? NP : NI;
+      LIN(y->h1, W, l.in, nullptr, y->proj, ldp, ldp, W, 0);
+      if (split)
+        TRY(B200Q_PROF_GEMM, 2.0 * T * 2.0 * F * W,
+            b200q_gemm_clamped_glu_bf16(y->h1, (const uint8_t*)l.in + (size_t)NP * W * es, l.in_b + NP, act, KO, T, 2 * F, W,
+                                        d.ff_limit, stream));
+      else if (F > 0)
+        TRY(EW, 3.0 * T * F * es,
+            b200q_clamped_glu_ex((uint8_t*)y->proj + (size_t)NP * es, ldp, l.in_b + NP, act, KO, T, F,
+                                 l.gate_up_il ? 128 : 0, d.ff_limit, dt, stream));
+      // cosines and sines once per step for all layers of equal rotation
+      const b200q_layer_desc* td = rot_layer < 0 ? nullptr : &y->layers[rot_layer].d;
+      if (d.rot_dims > 0 && !(td && td->rot_dims == d.rot_dims && td->rot_base == d.rot_base && td->rot_factor == d.rot_factor &&
+                              td->rot_original == d.rot_original && td->rot_fast == d.rot_fast && td->rot_slow == d.rot_slow)) {
+        TRY(EW, 8.0 * T * d.rot_dims / 2, b200q_rot_table(l.freq, l.mag, b->positions, T, d.rot_dims / 2, y->rot, stream));
+        rot_layer = li;
+      }
+      uint8_t* cache = m->kv + m->num_blocks * l.cache_block_off;  // a borrowing layer's offset is the lender's
+      TRY(EW, (double)T * NC * 2 * es,
+          b200q_diff_attn_prep(y->proj, ldp, l.in_b, l.conv_w, d.conv_taps, d.conv_taps > 1 ? y->state + l.conv_off : nullptr,
+                               y->state_slot_floats, own ? 1 : 0, H, G, d.dim, d.vdim, d.rot_dims, y->rot, d.attn_scale,
+                               b->seq_desc, b->row_seq, b->n_rows, b->slot_mapping, c.block_size, y->qa, cache, T, dt, stream));
+      TRY(B200Q_PROF_DECODE_ATTN, (double)b->sum_ctx_dec * G * (2 * d.dim + d.vdim) * es,
+          b200q_diff_attn(y->qa, cache, b->block_table, b->bt_stride, b->row_seq, b->positions, b->seq_desc, b->n_rows, T, H,
+                          G, d.dim, d.vdim, c.block_size, l.map_lambda, 1.f - d.diff, c.rms_eps,
+                          (uint8_t*)y->proj + (size_t)NC * es, ldp, y->attn, KO, dt, stream));
+      // the output and down projections as one product over [heads | unit]; where it splits its reduction the closing
+      // sum adds the parts
+      const float* parts = nullptr;
+      int splits = 1;
+      if (dt == B200Q_DTYPE_BF16 && W % 64 == 0 && KO % 64 == 0 && m->fuse_splitk &&
+          ((reinterpret_cast<uintptr_t>(y->attn) | reinterpret_cast<uintptr_t>(l.out)) & 15) == 0)
+        TRY(B200Q_PROF_GEMM, 2.0 * T * (double)W * KO,
+            b200q_gemm_bf16_splitk(y->attn, l.out, T, W, KO, stream, &parts, &splits));
+      if (splits == 1) LIN(y->attn, KO, l.out, nullptr, y->mix, W, W, KO, 0);
+      const bool last = li + 1 == c.n_layers;
+      TRY(EW, (double)T * W * (8 + 2 * es),
+          b200q_layer_close(y->x, splits > 1 ? (const void*)parts : y->mix, splits > 1 ? 1 : 0, splits, l.out_b,
+                            last ? nullptr : y->layers[li + 1].norm1, last ? nullptr : y->h1, T, W, c.rms_eps, dt, stream));
       if (y->tap) TRY(EW, 8.0 * T * W, b200q_copy_f32(y->x, y->tap + (int64_t)li * T * W, (int64_t)T * W, stream));
       continue;
     }

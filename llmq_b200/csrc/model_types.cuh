@@ -44,6 +44,9 @@ struct b200q_layered_layer {
   // the gated GELU feed-forward (gate_up = [gate | up] rows), the per-layer token input; biases of window attention
   const float *norm1b = nullptr, *norm2b = nullptr, *proj_b = nullptr, *o_b = nullptr, *tok_norm = nullptr;
   const void *gate_up = nullptr, *tok_gate = nullptr, *tok_proj = nullptr;
+  // parallel form with a shared norm: fused projections of both sublayers, their biases, differential attention's factor
+  const void *in = nullptr, *out = nullptr;
+  const float *in_b = nullptr, *out_b = nullptr, *map_lambda = nullptr;
   float mag = 1.f;  // factor of sine and cosine (YaRN)
   bool gate_up_il = false;  // gate_up rows interleaved in blocks of 128 (the fused product + gated unit's layout)
   std::vector<b200q_layered_layer> side;  // the mixer beside the first one (none or one)
@@ -81,6 +84,7 @@ struct b200q_layered {
   const void* tok_embed = nullptr;
   int64_t tok_cols = 0;
   void *tg = nullptr, *ta = nullptr;
+  float* rot = nullptr;  // cosines and sines of the step's positions, shared by layers of equal rotation
 };
 
 struct b200q_layer {

@@ -62,6 +62,7 @@ class ModelConfig(C.Structure):
         ("residual_mult", C.c_float),
         ("side_dim", C.c_int32),
         ("logit_scale", C.c_float),
+        ("shared_norm", C.c_int32),
     ]
 
 
@@ -71,6 +72,7 @@ ARCH_RAMOPEL = 2
 ARCH_NORIDRA = 3
 ARCH_PALUZEN = 4
 ARCH_KABAVIK = 5
+ARCH_LIPEDRA = 6
 FORM_PARALLEL = 0
 FORM_POSTNORM = 1
 FORM_PRENORM = 2
@@ -89,6 +91,7 @@ MIXER_SELECTIVE_SCAN = 5
 MIXER_LIGHTNING = 6
 MIXER_WINDOW_ATTN = 7
 MIXER_DECAY_MIX = 8
+MIXER_DIFF_ATTN = 9
 FF_NONE = 0
 FF_POLYNORM = 1
 FF_MOE = 2
@@ -96,6 +99,7 @@ FF_MOE_SIGMOID = 3
 FF_RELU2 = 4
 FF_MOE_GROUPED = 5
 FF_GEGLU = 6
+FF_CLAMPED = 7
 
 
 class LayerDesc(C.Structure):
@@ -113,6 +117,7 @@ class LayerDesc(C.Structure):
         ("keep_first", C.c_int32), ("qk_norm", C.c_int32), ("proj_bias", C.c_int32), ("bare", C.c_int32),
         ("head_gate", C.c_int32), ("q_temp_coef", C.c_float), ("q_temp_every", C.c_int32),
         ("rot_factor", C.c_double), ("rot_original", C.c_double), ("rot_fast", C.c_double), ("rot_slow", C.c_double),
+        ("diff", C.c_float), ("ff_limit", C.c_float),
     ]
 
 
@@ -278,6 +283,17 @@ SIGNATURES = {
     "b200q_latent_prep_ex": (_i, [_vp, _i, _i, _i, _i, _i, _vp, _f, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _f, _i, _vp]),
     "b200q_rope_pairs_q_ex": (_i, [_vp, _i, _i, _i, _i, _i, _vp, _f, _vp, _vp, _i, _i, _i, _vp]),
     "b200q_latent_attn_ex": (_i, [_vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _vp, _i, _vp, _i, _vp]),
+    # parallel layers with one shared norm, differential attention
+    "b200q_layer_close": (_i, [_vp, _vp, _i, _i, _vp, _vp, _vp, _i, _i, _f, _i, _vp]),
+    "b200q_clamped_glu_ex": (_i, [_vp, _i, _vp, _vp, _i, _i64, _i, _i, _f, _i, _vp]),
+    "b200q_gemm_clamped_glu_bf16": (_i, [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _f, _vp]),
+    "b200q_rot_table": (_i, [_vp, _f, _vp, _i, _i, _vp, _vp]),
+    "b200q_diff_attn_tiled": (_i, [_i, _i, _i, _i]),
+    "b200q_diff_attn_prep": (_i, [_vp, _i, _vp, _vp, _i, _vp, _ll, _i, _i, _i, _i, _i, _i, _vp, _f, _vp, _vp, _i, _vp, _i, _vp,
+                                  _vp, _i, _i, _vp]),
+    "b200q_diff_attn": (_i, [_vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp, _f, _f, _vp, _i, _vp, _i, _i,
+                             _vp]),
+    "b200q_wait_failures": (_i, []),
     "b200q_model_create_layered": (_i, [C.POINTER(ModelConfig), C.POINTER(LayerDesc), C.POINTER(_vp)]),
     "b200q_model_kv_block_bytes": (_i64, [_vp]),
     "b200q_model_state_slot_bytes": (_i64, [_vp]),
