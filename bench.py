@@ -697,7 +697,9 @@ def run_compare(args):
         cache = state = 0
         for ly in spec.layers:
             kind = getattr(ly, "kind", None)        # Paluzen's layer runs (a repeated layer counts once per pass)
-            if kind in ("attention", "attention_2") and hasattr(ly, "keep_first"):   # Kabavik: window + kept first keys
+            if hasattr(ly, "diff"):                 # Lipedra: two key maps and one value per key head, every earlier key
+                cache += B * (C0 + 1) * ly.kv_heads * (2 * ly.dim + ly.vdim) * 2
+            elif kind in ("attention", "attention_2") and hasattr(ly, "keep_first"):   # Kabavik: window + kept first keys
                 seen = min(C0 + 1, ly.window + ly.keep_first) if ly.window else C0 + 1
                 cache += B * seen * ly.kv_heads * (ly.dim + ly.vdim) * 2
             elif kind == "latent_attention":
@@ -720,18 +722,20 @@ def run_compare(args):
         return cache, state
 
     def prefill_attention_flops(spec):
-        """score and value products of the cache-reading attention layers over the prefill workload (Kabavik's three
-        mixers, Paluzen's window attention)"""
+        """score and value products of the cache-reading attention layers over the prefill workload (Lipedra's two maps,
+        Kabavik's three mixers, Paluzen's window attention)"""
         fl = 0.0
         for ly in spec.layers:
             kind = getattr(ly, "kind", None)
-            if kind in ("attention", "attention_2", "parallel"):
+            if hasattr(ly, "diff"):
+                per_key = 2.0 * ly.heads * 2 * (ly.dim + ly.vdim)
+            elif kind in ("attention", "attention_2", "parallel"):
                 per_key = 2.0 * ly.heads * (ly.dim + ly.vdim)
             elif kind == "latent_attention" and hasattr(ly, "keep_first"):
                 per_key = 2.0 * ly.heads * (2 * ly.kv_rank + ly.rot_dim)
             else:
                 continue
-            w = ly.window or S_p
+            w = getattr(ly, "window", 0) or S_p
             keys = sum(min(p + 1, w) for p in range(S_p)) + getattr(ly, "keep_first", 0) * max(S_p - w, 0)
             fl += per_key * keys * n_p
         return fl
@@ -739,13 +743,16 @@ def run_compare(args):
     frac = lambda by, ms: round(by / (ms * 1e-3) / 1e9 / peaks["hbm_gbs"], 3) if ms > 0 else None
     tf = lambda fl, ms: round(fl / (ms * 1e-3) / 1e12 / peaks["bf16_tflops"], 3) if ms > 0 else None
     results = {}
-    if args.compare in ("noridra", "paluzen", "kabavik"):
+    if args.compare in ("noridra", "paluzen", "kabavik", "lipedra"):
         # the design beside the closest existing one at equal width and layer count: Noridra beside Ramopel
         # (layered, recurrent state slots, routed experts); Paluzen beside Noridra (windowed / chunked grouped-query
         # attention on the tensor cores, decayed outer-product states, routed experts)
         # Kabavik beside Paluzen (grouped-query window attention on the tensor cores, fp32 residual with fused sums and
         # norms, gated feed-forwards through the same GEMM)
-        new, old = args.compare, {"noridra": "ramopel", "paluzen": "noridra", "kabavik": "paluzen"}[args.compare]
+        # Lipedra beside Kabavik (grouped-query attention with biases over a paged cache, gated feed-forwards with the
+        # unit in the product's epilogue, borrowed keys and values)
+        new, old = args.compare, {"noridra": "ramopel", "paluzen": "noridra", "kabavik": "paluzen",
+                                  "lipedra": "kabavik"}[args.compare]
         for key in (args.compare_sizes or f"{new}-1b,{new}-3b").split(","):
             nspec, rspec = BUILTIN_SPECS[key], BUILTIN_SPECS[key.replace(new, old)]
             n, r = measure(nspec), measure(rspec)
@@ -837,11 +844,10 @@ def main():
     ap.add_argument("--cpu-budget-s", type=float, default=10.0)
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--dry-run", action="store_true", help="host-logic self-test without a GPU (not a measurement)")
-    ap.add_argument("--compare", default=None, choices=["ramopel", "noridra", "paluzen", "kabavik"],
+    ap.add_argument("--compare", default=None, choices=["ramopel", "noridra", "paluzen", "kabavik", "lipedra"],
                     help="instead of the headline workload: prefill / decode throughput of this design beside the closest "
-                         "existing model of equal size (ramopel: a Llama decoder; noridra: Ramopel; paluzen: Noridra; kabavik: Paluzen), random "
-                         "weights, one "
-                         "JSON line")
+                         "existing model of equal size (ramopel: a Llama decoder; noridra: Ramopel; paluzen: Noridra; kabavik: Paluzen; "
+                         "lipedra: Kabavik), random weights, one JSON line")
     ap.add_argument("--compare-sizes", default=None, help="builtin sizes, default <design>-1b,<design>-3b")
     ap.add_argument("--compare-prompt", type=int, default=2048)
     ap.add_argument("--compare-prompts", type=int, default=4)
