@@ -543,18 +543,20 @@ int b200q_diff_attn_tiled(int dim, int vdim, int block_size, int dtype);
  * indexed like a row; NULL: none); y_t = sum_j conv[j][c] u_(t - taps + 1 + j) (conv: fp32 [taps][channels], taps 0: off;
  * zeros before the sequence's start; the last taps - 1 values u travel in `state`, fp32 [taps - 1][channels]); of q and k
  * the pairs (2i, 2i + 1) of a map's first rot_dims dimensions are turned by `table` (b200q_rot_table).  q: [T, heads, 2,
- * dim] as b200q_diff_attn_tiled says; cache: [block][kv_heads][block_size][2*dim + vdim] = [key 1 | key 2 | value]. */
+ * dim] as b200q_diff_attn_tiled says; cache: [block][kv_heads][block_size][2*dim + vdim] = [key 1 | key 2 | value].
+ * max_portion (here and below): most tokens any sequence brings to the step, 0 = unknown (it sizes the grid only). */
 int b200q_diff_attn_prep(const void* proj_dev, int ldp, const float* bias_dev, const float* conv_dev, int taps,
                          float* state_dev, long long slot_stride, int own, int heads, int kv_heads, int dim, int vdim,
                          int rot_dims, const float* table_dev, float scale, const int32_t* seq_desc_dev,
-                         const int32_t* row_seq_dev, int n_seqs, const int32_t* slot_mapping_dev, int block_size,
-                         void* q_dev, void* cache_dev, int T, int dtype, void* stream);
+                         const int32_t* row_seq_dev, int n_seqs, int max_portion, const int32_t* slot_mapping_dev,
+                         int block_size, void* q_dev, void* cache_dev, int T, int dtype, void* stream);
 /* differential attention 2/2: with a1, a2 the softmax attentions of a head's two maps over the keys j <= p of the token's
  * sequence, o = a1 - lambda a2 (lambda: one fp32 number), out[t, h*vdim ..] = o / sqrt(mean(o^2) + eps) * mult *
  * sigmoid(gate[t, h]) (gate NULL: 1); out rows of ld_out elements, gate rows of ld_gate */
 int b200q_diff_attn(const void* q_dev, const void* cache_dev, const int32_t* block_table_dev, int bt_stride,
                     const int32_t* row_seq_dev, const int32_t* positions_dev, const int32_t* seq_desc_dev, int n_seqs,
-                    int T, int heads, int kv_heads, int dim, int vdim, int block_size, const float* lambda_dev,
+                    int max_portion, int T, int heads, int kv_heads, int dim, int vdim, int block_size,
+                    const float* lambda_dev,
                     float mult, float eps, const void* gate_dev, int ld_gate, void* out_dev, int ld_out, int dtype,
                     void* stream);
 /* nonzero once a kernel's bounded wait has run out in this process (its outputs are then missing); engine steps report
@@ -801,6 +803,7 @@ typedef struct b200q_batch {
   const int32_t* seq_desc;      /* [n_rows][4]                                                   */
   const int32_t* row_seq;       /* [T]                                                           */
   int32_t no_sampling;          /* 1: stop after the logits (sample_rows may then hold up to max_logit_rows rows) */
+  int32_t max_portion;          /* most tokens any sequence brings to this step; 0 = unknown     */
 } b200q_batch;
 
 int b200q_model_create(const b200q_model_config* cfg, b200q_model_t* out);

@@ -140,9 +140,9 @@ __global__ void __launch_bounds__(256) diff_prep_state_kernel(DiffPrep a, int sk
 }
 
 // bf16, head sizes that are multiples of 8, up to 4 taps: a thread owns 8 neighbouring channels (whole rotated pairs)
-// and walks up to 16 consecutive tokens of a sequence with the last values in registers.  A single token's thread also
+// and walks up to 8 consecutive tokens of a sequence with the last values in registers.  A single token's thread also
 // stores the carried values itself: nobody else reads them.
-constexpr int PREP_TOKENS = 16;
+constexpr int PREP_TOKENS = 8;
 template <int TAPS>
 __global__ void __launch_bounds__(128) diff_prep_v8_kernel(DiffPrep a) {
   const int NQ = a.heads * 2 * a.dim, NK = a.own ? a.kv_heads * 2 * a.dim : 0, NV = a.own ? a.kv_heads * a.vdim : 0;
@@ -195,10 +195,17 @@ __global__ void __launch_bounds__(128) diff_prep_v8_kernel(DiffPrep a) {
   const int pairs = is_v ? 0 : max(0, min(4, (a.rot_dims - d) / 2));  // rotated pairs among the 8 channels
   const int cv = c - NQ - NK, ck = c - NQ;
   const int g = is_v ? cv / a.vdim : ck / (2 * a.dim), e = is_v ? 2 * a.dim + cv % a.vdim : ck % (2 * a.dim);
+  uint4 next = ld_v4(proj);
   for (int i = 0; i < n; ++i) {
     const long long t = s.row0 + r0 + i;
+    const uint32_t raw[4] = {next.x, next.y, next.z, next.w};
+    if (i + 1 < n) next = ld_v4(proj + (long long)(i + 1) * a.ldp);  // in flight while this token is worked on
     float u[8], y[8];
-    ldb8(proj + (long long)i * a.ldp, u);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      u[2 * k] = bf16_lo(raw[k]);
+      u[2 * k + 1] = bf16_hi(raw[k]);
+    }
 #pragma unroll
     for (int k = 0; k < 8; ++k) {
       u[k] += bias[k];
@@ -809,6 +816,12 @@ static int* wait_flag(int** dev) {
   return host;
 }
 
+// most tokens of a portion: what the caller says, or what a step of T tokens leaves for one of n_seqs sequences
+static int longest_portion(int max_portion, int n_seqs, int T) {
+  const int bound = T - n_seqs + 1;
+  return max_portion > 0 && max_portion < bound ? max_portion : bound;
+}
+
 static bool diff_attn_mma_mode() {  // B200Q_DIFF_ATTN_MMA=0: the scalar kernels everywhere
   static const bool on = [] {
     const char* v = getenv("B200Q_DIFF_ATTN_MMA");
@@ -818,18 +831,18 @@ static bool diff_attn_mma_mode() {  // B200Q_DIFF_ATTN_MMA=0: the scalar kernels
 }
 
 template <int DM, int VM>
-static int launch_diff_mma(const DiffAttn& a, int n_seqs, int T, cudaStream_t st) {
+static int launch_diff_mma(const DiffAttn& a, int n_seqs, int longest, int T, cudaStream_t st) {
   constexpr int STG = DM <= 64 ? 3 : 2, DSTG = DM <= 64 ? 3 : 2;
   const int RW = 2 * a.dim + a.vdim, rep = a.heads / a.kv_heads, parts = (rep + 7) / 8;
   if (T > n_seqs) {  // portions of prompts
-    const int ztiles = (T - n_seqs + 1 + 63) / 64;  // no portion of this step is longer than T - (n_seqs - 1)
-    dim3 grid(n_seqs, a.heads, ztiles);
+    dim3 grid(n_seqs, a.heads, (longest + 63) / 64);
     B200Q_CHECK_ARG(grid.y <= 65535 && grid.z <= 65535, "diff_attn: step too large (%d tokens)", T);
     const size_t smem = (size_t)STG * 64 * RW * 2 + (size_t)64 * ((2 * a.dim + 63) & ~63) * 2;
     auto kern = diff_attn_tile_kernel<DM, VM, STG>;
     if (smem > 48 * 1024) B200Q_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     kern<<<grid, 128, smem, st>>>(a, 1);
     B200Q_LAUNCH_CHECK();
+    if ((long long)n_seqs * longest == T) return B200Q_OK;  // every portion is as long: no single tokens
   }
   dim3 grid(n_seqs, a.kv_heads * parts);
   B200Q_CHECK_ARG(grid.y <= 65535, "diff_attn: too many heads");
@@ -868,7 +881,7 @@ int b200q_rot_table(const double* freq, float mag, const int32_t* positions, int
 int b200q_diff_attn_prep(const void* proj, int ldp, const float* bias, const float* conv, int taps, float* state,
                          long long slot_stride, int own, int heads, int kv_heads, int dim, int vdim, int rot_dims,
                          const float* table, float scale, const int32_t* seq_desc, const int32_t* row_seq, int n_seqs,
-                         const int32_t* slot_mapping, int block_size, void* q, void* cache, int T_, int dtype,
+                         int max_portion, const int32_t* slot_mapping, int block_size, void* q, void* cache, int T_, int dtype,
                          void* stream) {
   B200Q_CHECK_ARG(proj && q && seq_desc && row_seq && n_seqs > 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0 &&
                       dim > 0 && vdim > 0 && block_size > 0 && T_ >= 0 && is_dtype(dtype) &&
@@ -891,7 +904,7 @@ int b200q_diff_attn_prep(const void* proj, int ldp, const float* bias, const flo
                     reinterpret_cast<uintptr_t>(state) | reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache)) &
                    15) == 0;
   if (v8) {
-    dim3 grid(n_seqs, (C / 8 + 127) / 128, (T_ - n_seqs + 1 + PREP_TOKENS - 1) / PREP_TOKENS);
+    dim3 grid(n_seqs, (C / 8 + 127) / 128, (longest_portion(max_portion, n_seqs, T_) + PREP_TOKENS - 1) / PREP_TOKENS);
     B200Q_CHECK_ARG(grid.y <= 65535 && grid.z <= 65535, "diff_attn_prep: step too large (%d tokens)", T_);
     if (taps <= 1) diff_prep_v8_kernel<1><<<grid, 128, 0, st>>>(a);
     else if (taps == 2) diff_prep_v8_kernel<2><<<grid, 128, 0, st>>>(a);
@@ -913,8 +926,8 @@ int b200q_diff_attn_prep(const void* proj, int ldp, const float* bias, const flo
 }
 
 int b200q_diff_attn(const void* q, const void* cache, const int32_t* block_table, int bt_stride, const int32_t* row_seq,
-                    const int32_t* positions, const int32_t* seq_desc, int n_seqs, int T_, int heads, int kv_heads, int dim,
-                    int vdim, int block_size, const float* lambda, float mult, float eps, const void* gate, int ld_gate,
+                    const int32_t* positions, const int32_t* seq_desc, int n_seqs, int max_portion, int T_, int heads,
+                    int kv_heads, int dim, int vdim, int block_size, const float* lambda, float mult, float eps, const void* gate, int ld_gate,
                     void* out, int ld_out, int dtype, void* stream) {
   B200Q_CHECK_ARG(q && cache && block_table && row_seq && positions && seq_desc && n_seqs > 0 && lambda && out &&
                       heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && dim > 0 && dim <= 256 && vdim > 0 && vdim <= 512 &&
@@ -936,7 +949,8 @@ int b200q_diff_attn(const void* q, const void* cache, const int32_t* block_table
     B200Q_CHECK_ARG(((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache)) & 15) == 0 &&
                         (reinterpret_cast<uintptr_t>(out) & 3) == 0 && ld_out % 2 == 0,
                     "diff_attn: queries and cache must be 16-byte aligned, output rows 4-byte aligned");
-    return dim <= 64 ? launch_diff_mma<64, 128>(a, n_seqs, T_, st) : launch_diff_mma<128, 128>(a, n_seqs, T_, st);
+    const int longest = longest_portion(max_portion, n_seqs, T_);
+    return dim <= 64 ? launch_diff_mma<64, 128>(a, n_seqs, longest, T_, st) : launch_diff_mma<128, 128>(a, n_seqs, longest, T_, st);
   }
   dim3 grid(T_, kv_heads, (heads / kv_heads + 3) / 4);
   B200Q_CHECK_ARG(grid.y <= 65535 && grid.z <= 65535, "diff_attn: too many heads");

@@ -749,6 +749,8 @@ static int launch_step(b200q_engine* e, InFlightStep& step, std::vector<Request*
     b.prev_out_ids = e->d_out;  // the in-flight step's ids: read by this step's embedding before its sampler overwrites them
     b.sample_params = any_sampled ? e->d_meta + (sparams - h_meta) : nullptr;
     b.n_rows = n_rows;
+    b.max_portion = 0;
+    for (Request* r : sched) b.max_portion = std::max(b.max_portion, (int32_t)r->n_sched);
     b.seq_desc = e->d_meta + (sdesc - h_meta);
     b.row_seq = e->d_meta + (rseq - h_meta);
     b.no_sampling = replay ? 1 : 0;

@@ -1217,10 +1217,11 @@ int layered_forward(b200q_model* m, const b200q_batch* b, void* stream) {
       TRY(EW, (double)T * NC * 2 * es,
           b200q_diff_attn_prep(y->proj, ldp, l.in_b, l.conv_w, d.conv_taps, d.conv_taps > 1 ? y->state + l.conv_off : nullptr,
                                y->state_slot_floats, own ? 1 : 0, H, G, d.dim, d.vdim, d.rot_dims, y->rot, d.attn_scale,
-                               b->seq_desc, b->row_seq, b->n_rows, b->slot_mapping, c.block_size, y->qa, cache, T, dt, stream));
+                               b->seq_desc, b->row_seq, b->n_rows, b->max_portion, b->slot_mapping, c.block_size, y->qa, cache, T, dt,
+                               stream));
       TRY(B200Q_PROF_DECODE_ATTN, (double)b->sum_ctx_dec * G * (2 * d.dim + d.vdim) * es,
-          b200q_diff_attn(y->qa, cache, b->block_table, b->bt_stride, b->row_seq, b->positions, b->seq_desc, b->n_rows, T, H,
-                          G, d.dim, d.vdim, c.block_size, l.map_lambda, 1.f - d.diff, c.rms_eps,
+          b200q_diff_attn(y->qa, cache, b->block_table, b->bt_stride, b->row_seq, b->positions, b->seq_desc, b->n_rows,
+                          b->max_portion, T, H, G, d.dim, d.vdim, c.block_size, l.map_lambda, 1.f - d.diff, c.rms_eps,
                           (uint8_t*)y->proj + (size_t)NC * es, ldp, y->attn, KO, dt, stream));
       // the output and down projections as one product over [heads | unit]; where it splits its reduction the closing
       // sum adds the parts

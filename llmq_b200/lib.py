@@ -144,6 +144,7 @@ class Batch(C.Structure):
         ("seq_desc", C.c_void_p),
         ("row_seq", C.c_void_p),
         ("no_sampling", C.c_int32),
+        ("max_portion", C.c_int32),
     ]
 
 
@@ -289,9 +290,9 @@ SIGNATURES = {
     "b200q_gemm_clamped_glu_bf16": (_i, [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _f, _vp]),
     "b200q_rot_table": (_i, [_vp, _f, _vp, _i, _i, _vp, _vp]),
     "b200q_diff_attn_tiled": (_i, [_i, _i, _i, _i]),
-    "b200q_diff_attn_prep": (_i, [_vp, _i, _vp, _vp, _i, _vp, _ll, _i, _i, _i, _i, _i, _i, _vp, _f, _vp, _vp, _i, _vp, _i, _vp,
-                                  _vp, _i, _i, _vp]),
-    "b200q_diff_attn": (_i, [_vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp, _f, _f, _vp, _i, _vp, _i, _i,
+    "b200q_diff_attn_prep": (_i, [_vp, _i, _vp, _vp, _i, _vp, _ll, _i, _i, _i, _i, _i, _i, _vp, _f, _vp, _vp, _i, _i, _vp, _i,
+                                  _vp, _vp, _i, _i, _vp]),
+    "b200q_diff_attn": (_i, [_vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _f, _f, _vp, _i, _vp, _i, _i,
                              _vp]),
     "b200q_wait_failures": (_i, []),
     "b200q_model_create_layered": (_i, [C.POINTER(ModelConfig), C.POINTER(LayerDesc), C.POINTER(_vp)]),

@@ -148,8 +148,8 @@ def _diff_op(cuda, q, k, v, lam, mult, eps, gate, scale, dtype, portions, block_
         table = bt if c else bt[1:].contiguous()
         out = torch.zeros(c + n, H * V + 8, dtype=tdt, device=cuda)
         L.check(lib.b200q_diff_attn(q_step.data_ptr(), cache.data_ptr(), table.data_ptr(), nb, row_seq.data_ptr(),
-                                    pos.data_ptr(), desc.data_ptr(), 1 + c, c + n, H, G, D, V, block_size, lamd.data_ptr(),
-                                    mult, eps, g_step.data_ptr(), H + 3, out.data_ptr(), H * V + 8, dtype, None))
+                                    pos.data_ptr(), desc.data_ptr(), 1 + c, n if at % 2 else 0, c + n, H, G, D, V,
+                                    block_size, lamd.data_ptr(), mult, eps, g_step.data_ptr(), H + 3, out.data_ptr(), H * V + 8, dtype, None))
         torch.cuda.synchronize()
         assert float(out[:, H * V:].float().abs().max()) == 0.0            # nothing behind the heads is touched
         if c:                                                              # its only key, gate 0: a half
@@ -281,8 +281,8 @@ def test_preparation_continues_across_portions(cuda, case, dtype, cuts):
         L.check(lib.b200q_diff_attn_prep(pr.data_ptr(), ld, bd.data_ptr(), cd.data_ptr() if taps else None, taps,
                                          state.data_ptr() if taps > 1 else None, stride, int(own), H, G, D, V, rd,
                                          tab.data_ptr() if rd else None, scale, descd.data_ptr(), rseqd.data_ptr(),
-                                         len(part), smapd.data_ptr(), bs, q.data_ptr(), cache.data_ptr() if own else None,
-                                         row, dt, None))
+                                         len(part), max(ns) if i % 2 else 0, smapd.data_ptr(), bs, q.data_ptr(),
+                                         cache.data_ptr() if own else None, row, dt, None))
         torch.cuda.synchronize()
         for r, s in enumerate(part):
             qs[s].append(q[desc[r][0]:desc[r][0] + ns[s]].float().cpu())
