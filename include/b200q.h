@@ -30,7 +30,7 @@
 extern "C" {
 #endif
 
-#define B200Q_VERSION 6
+#define B200Q_VERSION 7
 
 #define B200Q_OK 0
 #define B200Q_EINVAL (-1)   /* bad argument / unsupported shape            */
@@ -527,7 +527,7 @@ int b200q_layer_close(float* x_dev, const void* y_dev, int y_f32, int splits, co
  * columns side by side (block 0) or interleaved in blocks of `block` columns (block must divide F) */
 int b200q_clamped_glu_ex(const void* gate_up_dev, int ld_in, const float* bias_dev, void* y_dev, int ld_out, int64_t rows,
                          int F, int block, float limit, int dtype, void* stream);
-/* fused gate_up GEMM + clamped unit: C[M, N/2] (rows of ldc elements); weight rows and bias (fp32 [N]) interleaved in
+/* fused gate_up GEMM + clamped unit: C[M, N/2] (rows of ldc elements); weight rows and bias (fp32 [N], NULL: none) interleaved in
  * blocks of 128 as for b200q_gemm_swiglu_bf16; the unit works on the fp32 accumulators */
 int b200q_gemm_clamped_glu_bf16(const void* A_dev, const void* W_dev, const float* bias_dev, void* C_dev, int ldc, int M,
                                 int N, int K, float limit, void* stream);
@@ -559,6 +559,62 @@ int b200q_diff_attn(const void* q_dev, const void* cache_dev, const int32_t* blo
                     const float* lambda_dev,
                     float mult, float eps, const void* gate_dev, int ld_gate, void* out_dev, int ld_out, int dtype,
                     void* stream);
+/* ---- retention, softmax sinks, group-routed gated experts (retention.cu, options of the kernels above) ---------------- */
+
+/* retention over the sequences of a step.  proj rows (model dtype, stride ldp) = [q (heads*dim) | k (heads*dim) | v
+ * (heads*vdim) | gate (heads*vdim)]; the first rot_dims of every head's q and k are turned in pairs (i, i + rot_dims/2) by
+ * `table` (b200q_rot_table; NULL with rot_dims 0), k is multiplied by dim^-1/2;  S <- decay[h] S + k v^T;  o = S^T q;
+ * out[t, h*vdim ..] = o / sqrt(mean(o^2) + eps) * silu(gate).  state: fp32 [heads][dim][vdim] per slot.  scratch: fp32
+ * b200q_retention_scratch_floats(heads, dim, vdim) * T floats, needed when T > n_seqs.  Single tokens take one fused
+ * kernel; portions are prepared, then run token by token (fp32 models, other sizes) or, for bf16 and dim 64 or 128, in
+ * chunks of 64 tokens on the tensor cores (operands split into bf16 high and low parts, the state in fp32). */
+int64_t b200q_retention_scratch_floats(int heads, int dim, int vdim);
+int b200q_retention(const void* proj_dev, int ldp, int heads, int dim, int vdim, int rot_dims, const float* table_dev,
+                    const float* decay_dev, float* state_dev, long long slot_stride, const int32_t* seq_desc_dev,
+                    const int32_t* row_seq_dev, int n_seqs, int max_portion, float eps, float* scratch_dev, void* out_dev,
+                    int T, int dtype, void* stream);
+/* b200q_window_attn_prep_ex with the rotation from `table` (b200q_rot_table) instead of frequencies; no temperatures */
+int b200q_window_attn_prep_tab(const void* proj_dev, int ldp, int q_off, int k_off, int v_off, const float* bias_dev,
+                               int heads, int kv_heads, int dim, int vdim, int qk_norm, const float* w_qn_dev,
+                               const float* w_kn_dev, float eps, int rot_dims, const float* table_dev,
+                               const int32_t* slot_mapping_dev, float scale, float* qs_dev, void* cache_dev, int T,
+                               int dtype, void* stream);
+/* b200q_window_attn_ex with a softmax sink (fp32 [heads], NULL: none: the denominator also holds exp(sink[h])) and, with
+ * channel_gate, a gate value per output channel (gate rows of heads*vdim values instead of heads) */
+int b200q_window_attn_sink(const float* qs_dev, const void* cache_dev, const int32_t* block_table_dev, int bt_stride,
+                           const int32_t* row_seq_dev, const int32_t* positions_dev, const int32_t* seq_desc_dev,
+                           int n_seqs, int T, int heads, int kv_heads, int dim, int vdim, int block_size, int window,
+                           int keep_first, float softcap, const float* sink_dev, const void* gate_dev, int ld_gate,
+                           int channel_gate, void* out_dev, int dtype, void* stream);
+/* latent attention with full-rank queries, steps 1 and 2 in one: proj rows = [q (heads x [dim | rot_dim]) | latent
+ * (kv_rank) | shared rotated key (rot_dim)];  cache row slot_mapping[t] = [latent / rms * w_kvn | turned key],
+ * qa[t, h, kv_rank ..] = turned query part; pairs (i, i + rot_dims/2) of the first rot_dims, by `table` */
+int b200q_latent_prep_tab(const void* proj_dev, int ldp, int heads, int dim, int kv_rank, int rot_dim, int rot_dims,
+                          const float* table_dev, const int32_t* slot_mapping_dev, const float* w_kvn_dev, float* qa_dev,
+                          void* cache_dev, int T, float eps, int dtype, void* stream);
+/* b200q_latent_attn_ex with a softmax sink (fp32 [heads], NULL: none) */
+int b200q_latent_attn_sink(const float* qa_dev, const void* cache_dev, const int32_t* block_table_dev, int bt_stride,
+                           const int32_t* row_seq_dev, const int32_t* positions_dev, int T, int heads, int kv_rank,
+                           int rot_dim, int block_size, int window, float scale, const float* sink_dev,
+                           const void* gate_dev, int ld_gate, void* out_dev, int dtype, void* stream);
+/* routing of B200Q_FF_MOE_GATED over fp32 router logits [T, E]: s = sigmoid(logits), choice = s + correction; only experts
+ * of the keep best of n_groups groups (score: sum of the two largest choices of the group) may be chosen; the top largest
+ * choices (ties: lowest index) -> idx, wts = s.  shared 1: every token has one more pair, expert E with weight 1.  Outputs
+ * as in b200q_moe_route over E + shared groups and top + shared pairs per token. */
+int b200q_moe_route_gated(const float* logits_dev, const float* correction_dev, int T, int E, int top, int n_groups,
+                          int keep, int shared, int32_t* idx_dev, float* wts_dev, int32_t* group_off_dev,
+                          int32_t* perm_tok_dev, int32_t* pair_pos_dev, int32_t* tile_tab_dev, int32_t* n_tiles_dev,
+                          void* stream);
+/* x[t] += y / sqrt(mean(y^2) + eps) * post_w, then (next_w) out[t] = x / sqrt(mean(x^2) + eps) * next_w in the model dtype.
+ * y = the sum over `splits` of fp32 [splits][T][W] (y_f32), the model-dtype rows y, or with pair_pos the sum over k < top
+ * of wts[t*top + k] * y[pair_pos[t*top + k]]; plus the model-dtype rows y2 (NULL: none) */
+int b200q_sandwich_close(float* x_dev, const void* y_dev, int y_f32, int splits, const int32_t* pair_pos_dev,
+                         const float* wts_dev, int top, const void* y2_dev, const float* post_w_dev,
+                         const float* next_w_dev, void* out_dev, int T, int W, float eps, int dtype, void* stream);
+/* x[t] += step (+ x0[t], x0 may be NULL); keep (fp32 [T, W] or NULL) receives x as it was; then out[t] = x / sqrt(mean(x^2)
+ * + eps) * w in the model dtype */
+int b200q_pass_begin(float* x_dev, const float* x0_dev, const float* step_dev, float* keep_dev, const float* w_dev,
+                     void* out_dev, int T, int W, float eps, int dtype, void* stream);
 /* nonzero once a kernel's bounded wait has run out in this process (its outputs are then missing); engine steps report
  * it as B200Q_ECUDA */
 int b200q_wait_failures(void);
@@ -648,6 +704,13 @@ typedef struct b200q_model_config {
  * head and optionally an earlier layer's keys and values; a clamped gated feed-forward with biases. */
 #define B200Q_ARCH_LIPEDRA 6
 
+/* Fimilorn: a layered decoder with an RMS norm on both sides of every sublayer (sandwich form) whose layers may run
+ * several times with the same weights; every pass begins with x <- x (+ x0) + step vector.  Retention, grouped-query
+ * attention with a softmax sink, norms over the whole query / key projection and a sigmoid gate per channel, latent
+ * attention with full-rank queries, a sliding window and a sink; clamped dense or group-routed gated experts; a tied
+ * output matrix. */
+#define B200Q_ARCH_FIMILORN 7
+
 #define B200Q_FORM_PARALLEL 0  /* x <- x + mixer(norm1 x) + ff(norm2 x)                                  */
 #define B200Q_FORM_POSTNORM 1  /* x <- norm1(alpha x + ls1 mixer(x~)); x <- norm2(alpha x + ls2 ff(x~)) */
 #define B200Q_FORM_PRENORM 2   /* x <- x + a mixer(h) (+ b side(h)), h = shift(norm1 x); x <- x + ff(norm2 x)     */
@@ -687,6 +750,10 @@ typedef struct b200q_model_config {
  * o / rms(o) * (1 - diff) * sigmoid(gate number of the head); q, k, v have biases and pass a causal convolution of
  * conv_taps taps per channel before the leading rot_dims of every map are turned (pairs 2i, 2i+1)             */
 #define B200Q_MIXER_DIFF_ATTN 9
+/* retention: linear attention with a constant decay per head over rotated queries and keys (pairs (i, i + rot_dims/2) of
+ * the first rot_dims of `dim`), keys times dim^-1/2;  S <- decay_h S + k v^T, o = S^T q, every head's o / rms(o), the
+ * concatenated heads times silu(gate)                                                                         */
+#define B200Q_MIXER_RETENTION 10
 #define B200Q_FF_NONE 0
 #define B200Q_FF_POLYNORM 1         /* down(PolyNorm(up h))                                                          */
 #define B200Q_FF_MOE 2              /* top-k of clamped gated experts + an optional gated shared expert              */
@@ -703,7 +770,18 @@ typedef struct b200q_model_config {
                                        of 128), which a bf16 model runs with the unit in the product's epilogue */
 
 #define B200Q_FF_CLAMPED 7          /* down(g' sigmoid(1.702 g') (u' + 1)), g' = min(gate h, ff_limit), u' = clamp(up h,
-                                       -ff_limit, ff_limit); all three projections have biases (shared-norm layers)  */
+                                       -ff_limit, ff_limit); all three projections have biases in shared-norm layers,
+                                       none in the sandwich form ("mlp.gate_up" / "mlp.gate_up_il", "mlp.down")      */
+/* top-k of silu(gate h) * up h experts by sigmoid score: the choice adds a per-expert correction to the score and is
+ * limited to the best `keep_groups` of `n_groups` equal groups of neighbouring experts (a group's score = the sum of its
+ * two largest choice scores); weights = the chosen scores without correction, not renormalised, applied to the expert's
+ * OUTPUT; a shared expert (shared_dim > 0) runs for every token and is added                                      */
+#define B200Q_FF_MOE_GATED 8
+
+#define B200Q_INJECT_NONE 0
+#define B200Q_INJECT_MATRIX 1       /* pre-norm form: x <- W_in [x; x0] ("inject" [W, 2W]; x0 = the embedding output)  */
+#define B200Q_INJECT_STEP 2         /* sandwich form: x <- x + s ("step" [1, W])                                      */
+#define B200Q_INJECT_STEP_EMBED 3   /* sandwich form: x <- x + x0 + s                                                 */
 
 typedef struct b200q_layer_desc {
   int32_t mixer;        /* B200Q_MIXER_*                                                               */
@@ -735,7 +813,7 @@ typedef struct b200q_layer_desc {
   int32_t state_dim;    /* selective scan: state size per channel                                         */
   int32_t dt_rank;      /* selective scan: rank of the step-size projection                               */
   /* pre-norm form and mixers 6-8 (zero elsewhere) */
-  int32_t inject;       /* 1: before this layer x <- W_in [x; x0] ("inject" [W, 2W]; x0 = the embedding output) */
+  int32_t inject;       /* B200Q_INJECT_*: what happens to x before this layer                            */
   float mix_scale;      /* the mixer's output is multiplied by this (0 = 1)                               */
   int32_t n_identity;   /* grouped mixture: identity experts behind the n_experts real ones               */
   int32_t n_groups;     /* grouped mixture: groups of neighbouring experts (identity ones included)       */
@@ -768,6 +846,12 @@ typedef struct b200q_layer_desc {
   /* differential attention and the clamped feed-forward (zero elsewhere) */
   float diff;           /* differential attention: heads' outputs are multiplied by 1 - diff               */
   float ff_limit;       /* clamped feed-forward                                                            */
+  /* further options (zero = off) */
+  int32_t sink;         /* window / latent attention: the softmax's denominator also holds exp("mix.sink"[h]), a number
+                           per head without key and value, not scaled                                              */
+  int32_t channel_gate; /* window attention without temperature and gate numbers (bare): mix.proj gains heads*vdim
+                           gate rows behind the values; the heads' outputs are multiplied by their sigmoids           */
+  int32_t rot_half;     /* latent attention: pairs (i, i + rot_dims/2) instead of (2i, 2i+1)               */
 } b200q_layer_desc;
 
 typedef struct b200q_model* b200q_model_t;
@@ -841,7 +925,18 @@ int b200q_model_create(const b200q_model_config* cfg, b200q_model_t* out);
  *   projections: "in" [NP + 2*ff, W] = rows q | k | v (own keys and values) | gate numbers | zero rows up to NP, then
  *   gate | up rows of the feed-forward ("in_il": interleaved in blocks of 128, ff a multiple of 128); "in_b" [1, NP +
  *   2*ff] their biases in the same order; "out" [W, heads*vdim + ff] = [output projection | down projection]; "out_b"
- *   [1, W] (with a feed-forward).  NP is a multiple of 256 from 1024 used rows up, else of 64. */
+ *   [1, W] (with a feed-forward).  NP is a multiple of 256 from 1024 used rows up, else of 64.
+ * B200Q_ARCH_FIMILORN (cfg.layer_form = B200Q_FORM_SANDWICH, cfg.norm_kind = B200Q_NORM_RMS): per layer "norm1", "norm1b"
+ *   (and "norm2", "norm2b" with a feed-forward) [1, W], "step" [1, W] where a pass begins, and
+ *   retention: "mix.proj" [roundup64(2*heads*dim + 2*heads*vdim), W] (rows: q, k, v, gate), "mix.decay" [1, heads], "mix.o"
+ *   window attention (bare, channel_gate, qk_norm 1, sink): "mix.proj" [roundup64(q + k + v + gate rows), W],
+ *     "mix.q_norm" [1, heads*dim], "mix.k_norm" [1, kv_heads*dim], "mix.sink" [1, heads], "mix.o"
+ *   latent attention (q_rank 0, sink): "mix.down" [roundup64(q rows + kv_rank + rot_dim), W], "mix.kv_norm", "mix.sink",
+ *     "mix.uk_t", "mix.uv", "mix.o"
+ *   clamped ff: "mlp.gate_up" or "mlp.gate_up_il" [2*ff, W], "mlp.down"
+ *   gated experts: "mlp.router" [E, W], "mlp.router_bias" [1, E] (the correction), "mlp.experts_gate_up" [N*2*ff, W],
+ *     "mlp.experts_down" [N*W, ff]; a shared expert as large as the others is expert E of these stacks (N = E + 1), one
+ *     of another size has "mlp.shared_gate_up" [2*shared_dim, W] and "mlp.shared_down" [W, shared_dim] (N = E) */
 int b200q_model_create_layered(const b200q_model_config* cfg, const b200q_layer_desc* layers,
                                b200q_model_t* out);
 /* layered models: bytes of one cache block over all layers that own a latent cache (the caller allocates

@@ -126,8 +126,8 @@ constexpr int EPI_SMEM_PER_WARP = 32 * 128;  // 32 rows x 64 bf16
 // kAct: 0 = plain GEMM, 1 = SwiGLU (Llama), 2 = GeGLU with the tanh approximation (Gemma-2):
 // out = bf16(bf16(gelu_tanh(bf16(g))) * bf16(u)), gelu_tanh evaluated in fp32 like torch's kernel:
 // 0.5 * g * (1 + tanh(sqrt(2/pi) * (g + 0.044715 g^3)))
-// 3 = clamped unit with biases (Lipedra): g' sigmoid(1.702 g') (u' + 1), g' = min(g + bg, limit), u' = clamp(u + bu,
-// -limit, limit), in fp32 from the accumulators (one rounding); bias: fp32, this tile's [gate (BN/2) | up (BN/2)]
+// 3 = clamped unit (Lipedra: with biases; Fimilorn: without): g' sigmoid(1.702 g') (u' + 1), g' = min(g + bg, limit), u' = clamp(u + bu,
+// -limit, limit), in fp32 from the accumulators (one rounding); bias: fp32, this tile's [gate (BN/2) | up (BN/2)], or NULL
 constexpr int ACT_NONE = 0, ACT_SWIGLU = 1, ACT_GEGLU = 2, ACT_CLAMPED = 3;
 struct GateArgs {
   const float* bias;
@@ -181,7 +181,8 @@ __device__ __forceinline__ void epilogue_rows(uint32_t taddr, bf16* ctile, long 
           };
 #pragma unroll
           for (int j = 0; j < 8; ++j) {
-            const float4 x = __ldg(bg + j), y = __ldg(bu + j);
+            const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+            const float4 x = gate_bias ? __ldg(bg + j) : zero, y = gate_bias ? __ldg(bu + j) : zero;
             v[4 * j + 0] = unit(v[4 * j + 0], u[4 * j + 0], x.x, y.x);
             v[4 * j + 1] = unit(v[4 * j + 1], u[4 * j + 1], x.y, y.y);
             v[4 * j + 2] = unit(v[4 * j + 2], u[4 * j + 2], x.z, y.z);
@@ -369,7 +370,7 @@ __global__ void __launch_bounds__(GEMM_THREADS, 1)
         }
       } else {
         epilogue_rows<BN, kAct>(taddr, ctile, ldc, row0, M, epi_smem + (warp - 2) * EPI_SMEM_PER_WARP, lane,
-                                kAct == ACT_CLAMPED ? gate.bias + (long long)n_blk * BN : nullptr, gate.limit);
+                                kAct == ACT_CLAMPED && gate.bias ? gate.bias + (long long)n_blk * BN : nullptr, gate.limit);
       }
       tc_fence_before();
       __syncwarp();
@@ -614,7 +615,7 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(GEMM_THREADS, 1)
       bf16* ctile = C + (long long)row0 * ldc + (long long)n_blk * OUT_BN;
       const uint32_t taddr = tmem_base + ((uint32_t)(quarter * 32) << 16) + (uint32_t)(acc * BN);
       epilogue_rows<BN, kAct>(taddr, ctile, ldc, row0, M, epi_smem + (warp - 2) * EPI_SMEM_PER_WARP, lane,
-                                kAct == ACT_CLAMPED ? gate.bias + (long long)n_blk * BN : nullptr, gate.limit);
+                                kAct == ACT_CLAMPED && gate.bias ? gate.bias + (long long)n_blk * BN : nullptr, gate.limit);
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive_cluster(mapa_shared(tmem_empty + acc, 0));
@@ -1319,10 +1320,10 @@ int b200q_gemm_geglu_bf16(const void* A, const void* W, void* C, int M, int N, i
   return gemm_gated<ACT_GEGLU>("gemm_geglu", A, W, C, M, N, K, stream);
 }
 
-// the clamped gated unit with biases in the same epilogue; C has rows of ldc elements
+// the clamped gated unit (with biases unless NULL) in the same epilogue; C has rows of ldc elements
 int b200q_gemm_clamped_glu_bf16(const void* A, const void* W, const float* bias, void* C, int ldc, int M, int N, int K,
                                 float limit, void* stream) {
-  B200Q_CHECK_ARG(bias && ldc >= N / 2 && ldc % 8 == 0 && (reinterpret_cast<uintptr_t>(bias) & 15) == 0 && limit >= 0.f,
+  B200Q_CHECK_ARG(ldc >= N / 2 && ldc % 8 == 0 && (reinterpret_cast<uintptr_t>(bias) & 15) == 0 && limit >= 0.f,
                   "gemm_clamped_glu: bad bias, row stride (%d) or limit", ldc);
   return gemm_gated<ACT_CLAMPED>("gemm_clamped_glu", A, W, C, M, N, K, stream, ldc, GateArgs{bias, limit});
 }

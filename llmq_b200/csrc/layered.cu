@@ -37,6 +37,19 @@ b200q_layer_desc side_desc(const b200q_layer_desc& d) {
   return s;
 }
 
+// sandwich layers with RMS norms on both sides and nothing else in their sums: the closing sums take split-K parts and routed
+// experts directly, rotations read the step's tables
+bool rms_sandwich(const b200q_model_config& c) {
+  return c.layer_form == B200Q_FORM_SANDWICH && c.norm_kind == B200Q_NORM_RMS && c.side_dim == 0 &&
+         (c.residual_mult == 0.f || c.residual_mult == 1.f);
+}
+bool same_rotation(const b200q_layer_desc& a, const b200q_layer_desc& b) {
+  return a.rot_dims == b.rot_dims && a.rot_base == b.rot_base && a.rot_factor == b.rot_factor &&
+         a.rot_original == b.rot_original && a.rot_fast == b.rot_fast && a.rot_slow == b.rot_slow;
+}
+// experts in a gated mixture's stacked matrices: a shared expert as large as the others is one more
+bool shared_stacked(const b200q_layer_desc& d) { return d.ff == B200Q_FF_MOE_GATED && d.shared_dim == d.ff_dim; }
+
 int check_sequence_mixer(int i, const b200q_layer_desc& d) {
   if (d.mixer == B200Q_MIXER_LIGHTNING) {
     B200Q_CHECK_ARG(d.heads > 0 && d.dim > 0 && d.dim <= 256 && d.vdim > 0, "layer %d: bad lightning sizes (dim <= 256)", i);
@@ -54,6 +67,8 @@ int check_sequence_mixer(int i, const b200q_layer_desc& d) {
                         (d.bare || (d.proj_bias == 0 && d.qk_norm == 0 && d.q_temp_every == 0 && d.kv_from < 0)),
                     "layer %d: bad window-attention options (biases, query / key norms, a query temperature by "
                     "position and borrowed keys go with the bare projection layout)", i);
+    B200Q_CHECK_ARG((d.sink == 0 || d.sink == 1) && (d.channel_gate == 0 || (d.channel_gate == 1 && d.bare)),
+                    "layer %d: a gate per channel goes with the bare projection layout", i);
   }
   return B200Q_OK;
 }
@@ -61,7 +76,7 @@ int check_sequence_mixer(int i, const b200q_layer_desc& d) {
 int check_layered(const b200q_model_config* c, const b200q_layer_desc* L) {
   B200Q_CHECK_ARG(c && L, "layered config is null");
   B200Q_CHECK_ARG(c->arch == B200Q_ARCH_RAMOPEL || c->arch == B200Q_ARCH_NORIDRA || c->arch == B200Q_ARCH_PALUZEN ||
-                      c->arch == B200Q_ARCH_KABAVIK || c->arch == B200Q_ARCH_LIPEDRA,
+                      c->arch == B200Q_ARCH_KABAVIK || c->arch == B200Q_ARCH_LIPEDRA || c->arch == B200Q_ARCH_FIMILORN,
                   "create_layered: arch=%d is not a layered architecture", c->arch);
   B200Q_CHECK_ARG(c->layer_form == B200Q_FORM_PARALLEL || c->layer_form == B200Q_FORM_POSTNORM ||
                       c->layer_form == B200Q_FORM_PRENORM || c->layer_form == B200Q_FORM_SANDWICH,
@@ -92,9 +107,11 @@ int check_layered(const b200q_model_config* c, const b200q_layer_desc* L) {
                           d.q_rank >= 0 && d.kv_rank > 0 && d.kv_rank <= 1024 && d.window >= 0 && d.rot_dims >= 0 &&
                           d.rot_dims % 2 == 0 && d.rot_dims <= d.rot_dim && d.rot_factor >= 0.0 && d.rot_original >= 0.0,
                       "layer %d: bad latent attention sizes (kv_rank <= 1024, even rot.dims <= rot_dim)", i);
-      // full-rank queries (q_rank 0) and the gate number per head come as one fused projection of the layer's input
-      B200Q_CHECK_ARG((d.q_rank == 0) == (d.head_gate != 0) && (d.q_rank > 0 || d.kv_from < 0),
-                      "layer %d: full-rank queries (q_rank 0) come with a gate per head and latents of their own", i);
+      // full-rank queries (q_rank 0) and gate numbers per head come as one fused projection of the layer's input
+      B200Q_CHECK_ARG((d.q_rank == 0 ? d.kv_from < 0 : d.head_gate == 0) && (d.sink == 0 || d.sink == 1) &&
+                          (d.rot_half == 0 || (d.rot_half == 1 && d.q_rank == 0 && rms_sandwich(*c))),
+                      "layer %d: gates per head and half-split rotation go with full-rank queries (q_rank 0), those with "
+                      "latents of their own", i);
       if (d.kv_from >= 0) {
         B200Q_CHECK_ARG(d.kv_from < i && L[d.kv_from].mixer == B200Q_MIXER_LATENT_ATTN && L[d.kv_from].kv_from < 0 &&
                             L[d.kv_from].kv_rank == d.kv_rank && L[d.kv_from].rot_dim == d.rot_dim,
@@ -126,6 +143,12 @@ int check_layered(const b200q_model_config* c, const b200q_layer_desc* L) {
                         "layer %d: kv_from=%d must name an earlier window-attention layer with keys and values of its "
                         "own and the same sizes", i, d.kv_from);
       }
+    } else if (d.mixer == B200Q_MIXER_RETENTION) {
+      B200Q_CHECK_ARG(d.heads > 0 && d.dim > 0 && d.dim <= 256 && d.vdim > 0 && d.vdim <= 4096 && d.rot_dims >= 0 &&
+                          d.rot_dims % 2 == 0 && d.rot_dims <= d.dim && (d.rot_dims == 0 || d.rot_base > 0.0) &&
+                          rms_sandwich(*c),
+                      "layer %d: bad retention sizes (dim <= 256, vdim <= 4096, even rot.dims <= dim; sandwich layers with "
+                      "RMS norms)", i);
     } else if (d.mixer == B200Q_MIXER_DIFF_ATTN) {
       B200Q_CHECK_ARG(d.heads > 0 && d.kv_heads > 0 && d.heads % d.kv_heads == 0 && d.dim > 0 && d.dim <= 256 && d.vdim > 0 &&
                           d.vdim <= 512 && d.conv_taps >= 0 && d.conv_taps <= 16 && d.rot_dims >= 0 && d.rot_dims % 2 == 0 &&
@@ -149,16 +172,30 @@ int check_layered(const b200q_model_config* c, const b200q_layer_desc* L) {
                       "layer %d: side mixer %d is not one that can stand beside another", i, d.side_mixer);
       if (int rc = check_sequence_mixer(i, side_desc(d))) return rc;
     }
-    B200Q_CHECK_ARG((d.inject == 0 && d.side_mixer == 0 && d.mix_scale == 0.f) || c->layer_form == B200Q_FORM_PRENORM,
-                    "layer %d: re-injection, side mixers and mixer scales belong to the pre-norm form", i);
-    B200Q_CHECK_ARG(!sandwich || d.ff == B200Q_FF_GEGLU || d.ff == B200Q_FF_NONE,
+    B200Q_CHECK_ARG((d.side_mixer == 0 && d.mix_scale == 0.f) || c->layer_form == B200Q_FORM_PRENORM,
+                    "layer %d: side mixers and mixer scales belong to the pre-norm form", i);
+    B200Q_CHECK_ARG(d.inject == B200Q_INJECT_NONE ||
+                        (d.inject == B200Q_INJECT_MATRIX && c->layer_form == B200Q_FORM_PRENORM) ||
+                        ((d.inject == B200Q_INJECT_STEP || d.inject == B200Q_INJECT_STEP_EMBED) && rms_sandwich(*c)),
+                    "layer %d: re-injection %d does not go with this form of layers", i, d.inject);
+    B200Q_CHECK_ARG(!sandwich || d.ff == B200Q_FF_GEGLU || d.ff == B200Q_FF_NONE ||
+                        (rms_sandwich(*c) && (d.ff == B200Q_FF_CLAMPED || d.ff == B200Q_FF_MOE_GATED)),
                     "layer %d: feed-forward %d is not built for the sandwich form", i, d.ff);
-    B200Q_CHECK_ARG(!sandwich || d.mixer == B200Q_MIXER_LATENT_ATTN || d.mixer == B200Q_MIXER_WINDOW_ATTN,
+    B200Q_CHECK_ARG(!sandwich || d.mixer == B200Q_MIXER_LATENT_ATTN || d.mixer == B200Q_MIXER_WINDOW_ATTN ||
+                        d.mixer == B200Q_MIXER_RETENTION,
                     "layer %d: mixer %d is not built for the sandwich form", i, d.mixer);
     B200Q_CHECK_ARG(!c->shared_norm || (d.mixer == B200Q_MIXER_DIFF_ATTN && (d.ff == B200Q_FF_CLAMPED || d.ff == B200Q_FF_NONE)),
                     "layer %d: mixer %d / feed-forward %d are not built for layers with a shared norm", i, d.mixer, d.ff);
     if (d.ff == B200Q_FF_CLAMPED) {
-      B200Q_CHECK_ARG(d.ff_dim > 0 && d.ff_limit >= 0.f && c->shared_norm, "layer %d: bad clamped feed-forward", i);
+      B200Q_CHECK_ARG(d.ff_dim > 0 && d.ff_limit >= 0.f && (c->shared_norm || rms_sandwich(*c)),
+                      "layer %d: bad clamped feed-forward", i);
+    } else if (d.ff == B200Q_FF_MOE_GATED) {
+      B200Q_CHECK_ARG(d.ff_dim > 0 && d.n_experts > 0 && d.n_experts < 4095 && d.top_k > 0 && d.top_k < 32 && d.n_groups > 0 &&
+                          d.n_groups <= 256 && d.n_experts % d.n_groups == 0 && d.keep_groups > 0 &&
+                          d.keep_groups <= d.n_groups && d.top_k <= d.keep_groups * (d.n_experts / d.n_groups) &&
+                          d.shared_dim >= 0 && rms_sandwich(*c),
+                      "layer %d: bad gated mixture (experts < 4095, top < 32, at most 256 groups that divide the experts, top "
+                      "fits the kept groups)", i);
     } else if (d.ff == B200Q_FF_GEGLU) {
       B200Q_CHECK_ARG(d.ff_dim > 0 && sandwich, "layer %d: bad gated-GELU feed-forward", i);
     } else if (d.ff == B200Q_FF_RELU2) {
@@ -193,20 +230,21 @@ int check_layered(const b200q_model_config* c, const b200q_layer_desc* L) {
 struct Widths {
   int64_t proj = 1, cq = 1, q = 1, qa = 1, olat = 1, attn = 1, ffh = 1, ffa = 1, experts = 1, pairs = 1, egu = 1,
           eact = 1, delta = 0, cvf = 0, baf = 0, dtr = 0, xc = 0, xp = 0, blend = 0, rot = 0;
-  bool moe = false, shared = false, hf = false, side = false, inject = false;
+  bool moe = false, shared = false, hf = false, side = false, inject = false, keep_x0 = false;
 };
 int64_t pad64(int64_t v) { return (v + 63) & ~(int64_t)63; }
-// rows of window attention's fused projection: [q | k | v (own keys and values) | gate number per head (not bare)],
-// with zero rows up to a multiple of 64
+// rows of window attention's fused projection: [q | k | v (own keys and values) | gate number per head (not bare) or gate
+// value per channel], with zero rows up to a multiple of 64
 int64_t window_proj_rows(const b200q_layer_desc& d) {
   return pad64((int64_t)d.heads * d.dim + (d.kv_from < 0 ? (int64_t)d.kv_heads * (d.dim + d.vdim) : 0) +
-               (d.bare ? 0 : d.heads));
+               (d.bare ? 0 : d.heads) + (d.channel_gate ? (int64_t)d.heads * d.vdim : 0));
 }
 // rows of latent attention's fused projection with full-rank queries: [q | latent | shared rotated key | gate number
-// per head], with zero rows up to a multiple of 64
+// per head (head_gate)], with zero rows up to a multiple of 64
 int64_t latent_full_rows(const b200q_layer_desc& d) {
-  return pad64((int64_t)d.heads * (d.dim + d.rot_dim) + d.kv_rank + d.rot_dim + d.heads);
+  return pad64((int64_t)d.heads * (d.dim + d.rot_dim) + d.kv_rank + d.rot_dim + (d.head_gate ? d.heads : 0));
 }
+int64_t retention_proj_rows(const b200q_layer_desc& d) { return pad64(2 * (int64_t)d.heads * (d.dim + d.vdim)); }
 // channels of differential attention's q | k | v (k and v with own keys), and the rows of its part of the fused input
 // projection: those channels, a gate number per head, zero rows
 int64_t diff_channels(const b200q_layer_desc& d) {
@@ -275,6 +313,10 @@ Widths widths_of(const b200q_model_config& c, const std::vector<b200q_layered_la
       w.qa = std::max<int64_t>(w.qa, (int64_t)d.heads * 2 * d.dim);
       w.attn = std::max<int64_t>(w.attn, (int64_t)d.heads * d.vdim + clamped_ff(d));
       w.rot = std::max<int64_t>(w.rot, d.rot_dims);
+    } else if (d.mixer == B200Q_MIXER_RETENTION) {
+      w.proj = std::max<int64_t>(w.proj, retention_proj_rows(d));
+      w.cvf = std::max<int64_t>(w.cvf, b200q_retention_scratch_floats(d.heads, d.dim, d.vdim));
+      w.attn = std::max<int64_t>(w.attn, (int64_t)d.heads * d.vdim);
     } else {
       sequence_mixer_widths(d, c.hidden, w);
     }
@@ -282,7 +324,25 @@ Widths widths_of(const b200q_model_config& c, const std::vector<b200q_layered_la
       w.side = true;
       sequence_mixer_widths(side_desc(d), c.hidden, w);
     }
-    if (d.inject) w.inject = true;
+    if (d.inject == B200Q_INJECT_MATRIX) w.inject = w.keep_x0 = true;
+    if (d.inject == B200Q_INJECT_STEP_EMBED) w.keep_x0 = true;
+    w.rot = std::max<int64_t>(w.rot, l.rot_off + d.rot_dims);
+    if (d.ff == B200Q_FF_CLAMPED && c.layer_form == B200Q_FORM_SANDWICH) {
+      w.ffh = std::max<int64_t>(w.ffh, 2 * (int64_t)d.ff_dim);
+      w.ffa = std::max<int64_t>(w.ffa, d.ff_dim);
+    } else if (d.ff == B200Q_FF_MOE_GATED) {
+      const int64_t per = d.top_k + (shared_stacked(d) ? 1 : 0);
+      w.moe = true;
+      w.experts = std::max<int64_t>(w.experts, d.n_experts + 1);
+      w.pairs = std::max<int64_t>(w.pairs, per);
+      w.egu = std::max<int64_t>(w.egu, per * 2 * d.ff_dim);
+      w.eact = std::max<int64_t>(w.eact, per * d.ff_dim);
+      if (d.shared_dim > 0 && !shared_stacked(d)) {
+        w.shared = true;
+        w.ffh = std::max<int64_t>(w.ffh, 2 * (int64_t)d.shared_dim);
+        w.ffa = std::max<int64_t>(w.ffa, d.shared_dim);
+      }
+    }
     if (d.ff == B200Q_FF_GEGLU) {
       w.ffh = std::max<int64_t>(w.ffh, 2 * (int64_t)d.ff_dim);
       w.ffa = std::max<int64_t>(w.ffa, d.ff_dim);
@@ -365,7 +425,7 @@ int64_t layout(b200q_model* m, uint8_t* base) {
   y->shout = take(w.shared ? T * W * es : 1);
   y->sgate = (float*)take(T * 4);
   y->hf = (float*)take(w.hf ? T * W * 4 : 1);
-  y->x0 = (float*)take(w.inject ? T * W * 4 : 1);
+  y->x0 = (float*)take(w.keep_x0 ? T * W * 4 : 1);
   y->cat = take(w.inject ? T * 2 * W * es : 1);
   y->carry = (float*)take(c.token_shift ? (int64_t)c.max_seqs * W * 4 : 1);
   y->mix2 = take(w.side ? T * W * es : 1);
@@ -425,6 +485,13 @@ int layered_create(const b200q_model_config* cfg, const b200q_layer_desc* layers
         b200q_model_destroy(m);
         return rc;
       }
+    } else if (l.d.mixer == B200Q_MIXER_RETENTION) {
+      l.state_off = m->lay->state_slot_floats;
+      m->lay->state_slot_floats += (int64_t)l.d.heads * l.d.dim * l.d.vdim;
+      if ((rc = upload_frequencies(l))) {
+        b200q_model_destroy(m);
+        return rc;
+      }
     } else if (l.d.mixer == B200Q_MIXER_GENERAL_DELTA) {
       l.state_off = m->lay->state_slot_floats;
       m->lay->state_slot_floats += (int64_t)l.d.heads * l.d.dim * l.d.dim;
@@ -468,6 +535,17 @@ int layered_create(const b200q_model_config* cfg, const b200q_layer_desc* layers
         b200q_model_destroy(m);
         return rc;
       }
+    }
+    if (rms_sandwich(*cfg) && l.d.rot_dims > 0) {  // one table per distinct rotation, layers of equal rotation share it
+      l.rot_table = true;
+      l.rot_off = m->lay->rot_floats;
+      for (int j = 0; j < i; ++j)
+        if (m->lay->layers[j].rot_table && same_rotation(m->lay->layers[j].d, l.d)) {
+          l.rot_off = m->lay->layers[j].rot_off;
+          l.rot_shared = true;
+          break;
+        }
+      if (!l.rot_shared) m->lay->rot_floats += l.d.rot_dims;
     }
     if (l.d.side_mixer) {
       l.side.resize(1);
@@ -585,6 +663,7 @@ int layered_bind_weight(b200q_model* m, const char* name, const void* p, int64_t
       FIELD("tok.norm", l.tok_norm, 1, W)
     }
   }
+  if (d.inject == B200Q_INJECT_STEP || d.inject == B200Q_INJECT_STEP_EMBED) FIELD("step", l.step, 1, W)
   FIELD("norm1", l.norm1, 1, W)
   if (c.shared_norm) {
     const int64_t NI = diff_proj_rows(d) + 2 * clamped_ff(d);
@@ -605,7 +684,7 @@ int layered_bind_weight(b200q_model* m, const char* name, const void* p, int64_t
   }
   if (d.ff != B200Q_FF_NONE) FIELD("norm2", l.norm2, 1, W)
   if (c.token_shift) FIELD("shift", l.shift, 1, W)
-  if (d.inject) FIELD("inject", l.inject, W, 2 * W)
+  if (d.inject == B200Q_INJECT_MATRIX) FIELD("inject", l.inject, W, 2 * W)
   // the mixers of the pre-norm form, as a layer's first mixer ("mix.*") or beside it ("side.*")
   for (int which = 0; which < 2; ++which) {
     b200q_layered_layer* q = which == 0 ? &l : (l.side.empty() ? nullptr : &l.side[0]);
@@ -645,6 +724,11 @@ int layered_bind_weight(b200q_model* m, const char* name, const void* p, int64_t
         SUB("q_norm", q->q_norm, 1, e.qk_norm == 1 ? QD : e.dim)
         if (e.kv_from < 0) SUB("k_norm", q->kv_norm, 1, e.qk_norm == 1 ? (int64_t)e.kv_heads * e.dim : e.dim)
       }
+      if (e.sink) SUB("sink", q->sink, 1, e.heads)
+      SUB("o", q->o, W, QV)
+    } else if (e.mixer == B200Q_MIXER_RETENTION) {
+      SUB("proj", q->proj, retention_proj_rows(e), W)
+      SUB("decay", q->head_decay, 1, e.heads)
       SUB("o", q->o, W, QV)
     }
 #undef SUB
@@ -693,6 +777,7 @@ int layered_bind_weight(b200q_model* m, const char* name, const void* p, int64_t
       FIELD("mix.down", l.down, latent_full_rows(d), W)
     }
     if (d.kv_from < 0) FIELD("mix.kv_norm", l.kv_norm, 1, d.kv_rank)
+    if (d.sink) FIELD("mix.sink", l.sink, 1, d.heads)
     FIELD("mix.uk_t", l.uk_t, (int64_t)d.heads * d.kv_rank, d.dim)
     FIELD("mix.uv", l.uv, (int64_t)d.heads * d.vdim, d.kv_rank)
     FIELD("mix.o", l.o, W, (int64_t)d.heads * d.vdim)
@@ -704,7 +789,18 @@ int layered_bind_weight(b200q_model* m, const char* name, const void* p, int64_t
     FIELD("mix.out_norm", l.out_norm, 1, HD)
     FIELD("mix.o", l.o, W, HD)
   }
-  if (d.ff == B200Q_FF_GEGLU) {
+  if (d.ff == B200Q_FF_MOE_GATED) {
+    const int64_t N = d.n_experts + (shared_stacked(d) ? 1 : 0);
+    FIELD("mlp.router", l.router, d.n_experts, W)
+    FIELD("mlp.router_bias", l.router_bias, 1, d.n_experts)
+    FIELD("mlp.experts_gate_up", l.experts_gate_up, N * 2 * d.ff_dim, W)
+    FIELD("mlp.experts_down", l.experts_down, N * W, d.ff_dim)
+    if (d.shared_dim > 0 && !shared_stacked(d)) {
+      FIELD("mlp.shared_gate_up", l.shared_gate_up, 2 * (int64_t)d.shared_dim, W)
+      FIELD("mlp.shared_down", l.shared_down, W, d.shared_dim)
+    }
+  }
+  if (d.ff == B200Q_FF_GEGLU || (d.ff == B200Q_FF_CLAMPED && c.layer_form == B200Q_FORM_SANDWICH)) {
     FIELD("mlp.gate_up", l.gate_up, 2 * (int64_t)d.ff_dim, W)
     if (!strcmp(field, "mlp.gate_up_il")) {
       B200Q_CHECK_ARG(d.ff_dim % 128 == 0, "layer %d: interleaved gate / up rows need ff (%d) to be a multiple of 128", li,
@@ -771,6 +867,7 @@ static int check_bound(b200q_model* m) {
     }
     if (d.mixer == B200Q_MIXER_LATENT_ATTN) {
       need_kv = true;
+      ok = ok && (!d.sink || l.sink);
       ok = ok && l.down && (d.q_rank == 0 || (l.q_norm && l.uq)) && (d.kv_from >= 0 || l.kv_norm) && l.uk_t && l.uv;
     } else if (d.mixer == B200Q_MIXER_GENERAL_DELTA) {
       need_state = true;
@@ -789,24 +886,32 @@ static int check_bound(b200q_model* m) {
       need_state = true;
       ok = ok && l.shift;
     }
-    if (d.inject) ok = ok && l.inject;
+    if (d.inject == B200Q_INJECT_MATRIX) ok = ok && l.inject;
+    if (d.inject == B200Q_INJECT_STEP || d.inject == B200Q_INJECT_STEP_EMBED) ok = ok && l.step;
     for (const b200q_layered_layer* q : {&l, l.side.empty() ? (const b200q_layered_layer*)nullptr : &l.side[0]}) {
       if (!q) continue;
       if (q != &l) ok = ok && q->o;
       if (q->d.mixer == B200Q_MIXER_LIGHTNING) {
         need_state = true;
         ok = ok && q->proj && q->head_decay && q->out_norm;
+      } else if (q->d.mixer == B200Q_MIXER_RETENTION) {
+        need_state = true;
+        ok = ok && q->proj && q->head_decay;
       } else if (q->d.mixer == B200Q_MIXER_DECAY_MIX) {
         need_state = true;
         ok = ok && q->mu && q->proj && q->w1 && q->w2 && q->w0 && q->bonus && q->out_norm;
       } else if (q->d.mixer == B200Q_MIXER_WINDOW_ATTN) {
         need_kv = true;
+        ok = ok && (!q->d.sink || q->sink);
         ok = ok && q->proj && (q->d.bare || q->temp) && (!q->d.proj_bias || (q->proj_b && q->o_b)) &&
              (!q->d.qk_norm || (q->q_norm && (q->d.kv_from >= 0 || q->kv_norm)));
       }
     }
     if (d.ff == B200Q_FF_RELU2) ok = ok && l.up && l.ff_down;
-    if (d.ff == B200Q_FF_GEGLU) ok = ok && l.gate_up && l.ff_down;
+    if (d.ff == B200Q_FF_GEGLU || (d.ff == B200Q_FF_CLAMPED && !m->cfg.shared_norm)) ok = ok && l.gate_up && l.ff_down;
+    if (d.ff == B200Q_FF_MOE_GATED)
+      ok = ok && l.router && l.router_bias && l.experts_gate_up && l.experts_down &&
+           (d.shared_dim == 0 || shared_stacked(d) || (l.shared_gate_up && l.shared_down));
     if (m->cfg.layer_form == B200Q_FORM_SANDWICH)
       ok = ok && l.norm1b && (d.ff == B200Q_FF_NONE || l.norm2b) &&
            (m->cfg.side_dim == 0 || (l.tok_gate && l.tok_proj && l.tok_norm && m->lay->tok_embed));
@@ -874,6 +979,22 @@ int layered_forward(b200q_model* m, const b200q_batch* b, void* stream) {
         b200q_embed_f32(b->token_ids, b->prev_out_ids, m->embed, y->x, T, W, c.embed_scale > 0.f ? c.embed_scale : 1.f,
                         dt, stream));
 
+  // rms sandwich layers: a product whose reduction is split leaves its parts for the closing sum
+  const bool lean = rms_sandwich(c);
+  bool fold = false;  // the layer's closing sums can read parts
+  const float* parts = nullptr;
+  int splits = 1;
+  auto product = [&](const void* A, const void* Wt, void* outp, int K) -> int {  // [T, K] -> [T, W]
+    splits = 1;
+    if (fold && dt == B200Q_DTYPE_BF16 && W % 64 == 0 && K % 64 == 0 && m->fuse_splitk &&
+        ((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(Wt)) & 15) == 0)
+      TRY(B200Q_PROF_GEMM, 2.0 * T * (double)W * K, b200q_gemm_bf16_splitk(A, Wt, T, W, K, stream, &parts, &splits));
+    if (splits == 1) LIN(A, K, Wt, nullptr, outp, W, W, K, 0);
+    return B200Q_OK;
+  };
+  const float* rot0 = y->rot;  // a layer's table: rows of rot_dims values from rot_off * max_tokens
+  auto table_of = [&](const b200q_layered_layer& l) { return rot0 + l.rot_off * (int64_t)c.max_tokens; };
+
   // ---- mixers 6-8: read y->h1 [T, W] (model dtype; the decay mix reads the fp32 rows y->hf), write outp [T, W] ----
   auto run_sequence_mixer = [&](const b200q_layered_layer& l, void* outp) -> int {
     const b200q_layer_desc& d = l.d;
@@ -917,6 +1038,14 @@ int layered_forward(b200q_model* m, const b200q_batch* b, void* stream) {
           b200q_gated_rmsnorm(raw, HD, d.dim, l.out_norm, (uint8_t*)y->proj + (size_t)3 * HD * es, NQ, 1, c.rms_eps,
                               y->attn, T, dt, stream));
       LIN(y->attn, HD, l.o, nullptr, outp, W, W, HD, 0);
+    } else if (d.mixer == B200Q_MIXER_RETENTION) {
+      const int NP = (int)retention_proj_rows(d);
+      LIN(y->h1, W, l.proj, nullptr, y->proj, NP, NP, W, 0);  // [q | k | v | gate]
+      TRY(B200Q_PROF_PREFILL_ATTN, 4.0 * T * H * (double)d.dim * d.vdim,
+          b200q_retention(y->proj, NP, H, d.dim, d.vdim, d.rot_dims, table_of(l), l.head_decay, y->state + l.state_off,
+                          y->state_slot_floats, b->seq_desc, b->row_seq, b->n_rows, b->max_portion, c.rms_eps, y->cvf, y->attn,
+                          T, dt, stream));
+      return product(y->attn, l.o, outp, HV);
     } else {  // B200Q_MIXER_WINDOW_ATTN
       const int G = d.kv_heads, GD = G * d.dim, GV = G * d.vdim, NP = (int)window_proj_rows(d);
       const bool own = d.kv_from < 0;
@@ -924,7 +1053,12 @@ int layered_forward(b200q_model* m, const b200q_batch* b, void* stream) {
       uint8_t* cache = m->kv + m->num_blocks * l.cache_block_off;  // a borrowing layer's offset is the lender's
       // [q | k | v (own keys and values) | gate number per head (not bare) | zero rows]; biases join in the next step
       LIN(y->h1, W, l.proj, nullptr, y->proj, NP, NP, W, 0);
-      if (!d.bare && d.rot_factor == 0.0)
+      if (lean && d.bare && d.q_temp_every == 0)
+        TRY(EW, (double)T * ((HD + 2 * n_kv) * es + HD * 4),
+            b200q_window_attn_prep_tab(y->proj, NP, 0, own ? HD : -1, HD + GD, d.proj_bias ? l.proj_b : nullptr, H, G, d.dim,
+                                       d.vdim, d.qk_norm, l.q_norm, l.kv_norm, c.rms_eps, d.rot_dims, table_of(l),
+                                       b->slot_mapping, d.attn_scale, y->qa, cache, T, dt, stream));
+      else if (!d.bare && d.rot_factor == 0.0)
         TRY(EW, (double)T * ((HD + 2 * GD + 2 * GV) * es + HD * 4),
             b200q_window_attn_prep(y->proj, NP, H, G, d.dim, d.vdim, d.rot_dims, l.freq, b->positions, b->slot_mapping,
                                    l.temp, d.attn_scale, y->qa, cache, T, dt, stream));
@@ -935,10 +1069,12 @@ int layered_forward(b200q_model* m, const b200q_batch* b, void* stream) {
                                       b->positions, b->slot_mapping, d.bare ? nullptr : l.temp, d.attn_scale,
                                       d.q_temp_coef, d.q_temp_every, y->qa, cache, T, dt, stream));
       TRY(B200Q_PROF_DECODE_ATTN, (double)b->sum_ctx_dec * (GD + GV) * es,
-          b200q_window_attn_ex(y->qa, cache, b->block_table, b->bt_stride, b->row_seq, b->positions, b->seq_desc,
-                               b->n_rows, T, H, G, d.dim, d.vdim, c.block_size, d.window, d.keep_first, d.softcap,
-                               d.bare ? nullptr : (uint8_t*)y->proj + (size_t)(HD + n_kv) * es, NP, y->attn, dt, stream));
-      LIN(y->attn, HV, l.o, nullptr, outp, W, W, HV, 0);  // the output bias, if any, joins in the layer's sum
+          b200q_window_attn_sink(y->qa, cache, b->block_table, b->bt_stride, b->row_seq, b->positions, b->seq_desc,
+                                 b->n_rows, T, H, G, d.dim, d.vdim, c.block_size, d.window, d.keep_first, d.softcap,
+                                 d.sink ? l.sink : nullptr,
+                                 d.bare && !d.channel_gate ? nullptr : (uint8_t*)y->proj + (size_t)(HD + n_kv) * es, NP,
+                                 d.channel_gate, y->attn, dt, stream));
+      return product(y->attn, l.o, outp, HV);  // the output bias, if any, joins in the layer's sum
     }
     return B200Q_OK;
   };
@@ -946,7 +1082,8 @@ int layered_forward(b200q_model* m, const b200q_batch* b, void* stream) {
   // ---- the mixers: read y->h1 [T, W] (model dtype), write y->mix [T, W] ----
   auto run_mixer = [&](const b200q_layered_layer& l) -> int {
     const b200q_layer_desc& d = l.d;
-    if (d.mixer == B200Q_MIXER_LIGHTNING || d.mixer == B200Q_MIXER_DECAY_MIX || d.mixer == B200Q_MIXER_WINDOW_ATTN)
+    if (d.mixer == B200Q_MIXER_LIGHTNING || d.mixer == B200Q_MIXER_DECAY_MIX || d.mixer == B200Q_MIXER_WINDOW_ATTN ||
+        d.mixer == B200Q_MIXER_RETENTION)
       return run_sequence_mixer(l, y->mix);
     if (d.mixer == B200Q_MIXER_LATENT_ATTN) {
       const int R = d.kv_rank, P = d.rot_dim, RP = R + P, H = d.heads, QD = d.dim + P;
@@ -959,13 +1096,18 @@ int layered_forward(b200q_model* m, const b200q_batch* b, void* stream) {
         // full-rank queries: one projection of the layer's input gives [q | latent | shared rotated key | gates]
         const int nd = (int)latent_full_rows(d);
         LIN(y->h1, W, l.down, nullptr, y->proj, nd, nd, W, 0);
-        TRY(EW, (double)T * 2 * RP * es,
-            b200q_latent_prep_ex((uint8_t*)y->proj + (size_t)H * QD * es, nd, 0, R, P, d.rot_dims, l.freq, l.mag,
-                                 b->positions, b->slot_mapping, nullptr, l.kv_norm, nullptr, cache, 1, T, c.rms_eps, dt,
-                                 stream));
+        if (d.rot_half)
+          TRY(EW, (double)T * (2 * RP * es + H * P * (es + 4)),
+              b200q_latent_prep_tab(y->proj, nd, H, d.dim, R, P, d.rot_dims, table_of(l), b->slot_mapping, l.kv_norm, y->qa,
+                                    cache, T, c.rms_eps, dt, stream));
+        else
+          TRY(EW, (double)T * 2 * RP * es,
+              b200q_latent_prep_ex((uint8_t*)y->proj + (size_t)H * QD * es, nd, 0, R, P, d.rot_dims, l.freq, l.mag,
+                                   b->positions, b->slot_mapping, nullptr, l.kv_norm, nullptr, cache, 1, T, c.rms_eps, dt,
+                                   stream));
         q = y->proj;
         ldq = nd;
-        gate = (uint8_t*)y->proj + (size_t)(H * QD + RP) * es;
+        if (d.head_gate) gate = (uint8_t*)y->proj + (size_t)(H * QD + RP) * es;
       } else {
         const int nd = d.q_rank + (own ? RP : 0);
         LIN(y->h1, W, l.down, nullptr, y->proj, nd, nd, W, 0);
@@ -974,22 +1116,24 @@ int layered_forward(b200q_model* m, const b200q_batch* b, void* stream) {
                                  l.q_norm, l.kv_norm, y->cq, cache, own ? 1 : 0, T, c.rms_eps, dt, stream));
         LIN(y->cq, d.q_rank, l.uq, nullptr, y->q, H * QD, H * QD, d.q_rank, 0);
       }
-      TRY(EW, (double)T * H * P * (es + 4),
-          b200q_rope_pairs_q_ex(q, ldq, H, d.dim, P, d.rot_dims, l.freq, l.mag, b->positions, y->qa, R, T, dt, stream));
+      if (!d.rot_half)
+        TRY(EW, (double)T * H * P * (es + 4),
+            b200q_rope_pairs_q_ex(q, ldq, H, d.dim, P, d.rot_dims, l.freq, l.mag, b->positions, y->qa, R, T, dt, stream));
       // the unrotated query of every head, carried into the latent space: qa[t,h,:R] = W_uk[h]^T q[t,h,:dim]
       if (d.dim > 0)
         TRY(B200Q_PROF_GEMM, 2.0 * T * H * (double)R * d.dim,
             b200q_linear_batched(q, ldq, QD, l.uk_t, (long long)R * d.dim, y->qa, H * RP, RP, T, R, d.dim, H, dt, 1,
                                  stream));
       else
-        B200Q_CUDA(cudaMemsetAsync(y->qa, 0, (size_t)T * H * RP * 4, cst));
+        B200Q_CUDA(cudaMemset2DAsync(y->qa, (size_t)RP * 4, 0, (size_t)R * 4, (size_t)T * H, cst));
       TRY(B200Q_PROF_DECODE_ATTN, 0.0,
-          b200q_latent_attn_ex(y->qa, cache, b->block_table, b->bt_stride, b->row_seq, b->positions, T, H, R, P,
-                               c.block_size, d.window, d.attn_scale, gate, ldq, y->olat, dt, stream));
+          b200q_latent_attn_sink(y->qa, cache, b->block_table, b->bt_stride, b->row_seq, b->positions, T, H, R, P,
+                                 c.block_size, d.window, d.attn_scale, d.sink ? l.sink : nullptr, gate, ldq, y->olat, dt,
+                                 stream));
       TRY(B200Q_PROF_GEMM, 2.0 * T * H * (double)R * d.vdim,
           b200q_linear_batched(y->olat, H * R, R, l.uv, (long long)d.vdim * R, y->attn, H * d.vdim, d.vdim, T, d.vdim, R,
                                H, dt, 0, stream));
-      LIN(y->attn, H * d.vdim, l.o, nullptr, y->mix, W, W, H * d.vdim, 0);
+      return product(y->attn, l.o, y->mix, H * d.vdim);
     } else if (d.mixer == B200Q_MIXER_GENERAL_DELTA) {
       const int HD = d.heads * d.dim, NP = 5 * HD + d.decay_rank;
       LIN(y->h1, W, l.proj, nullptr, y->proj, NP, NP, W, 0);
@@ -1064,9 +1208,44 @@ int layered_forward(b200q_model* m, const b200q_batch* b, void* stream) {
     return B200Q_OK;
   };
 
+  // ---- gated experts of the sandwich form: read y->h2, leave the pairs' outputs in y->eout (and the shared expert's, if it is
+  // not one of them, in y->shout) ----
+  auto run_moe_gated = [&](const b200q_layered_layer& l) -> int {
+    const b200q_layer_desc& d = l.d;
+    const bool stacked = shared_stacked(d);
+    const int E = d.n_experts, N = E + (stacked ? 1 : 0), K = d.top_k + (stacked ? 1 : 0), F = d.ff_dim, P = T * K;
+    LIN(y->h2, W, l.router, nullptr, y->rlog, E, E, W, 1);
+    TRY(EW, (double)T * E * 4,
+        b200q_moe_route_gated(y->rlog, l.router_bias, T, E, d.top_k, d.n_groups, d.keep_groups, stacked ? 1 : 0, y->idx, y->wts,
+                              y->group_off, y->perm_tok, y->pair_pos, y->tile_tab, y->n_tiles, stream));
+    const bool sorted = dt == B200Q_DTYPE_BF16 && W % 8 == 0;
+    if (sorted) TRY(EW, 2.0 * P * W * es, b200q_gather_rows(y->h2, y->perm_tok, y->esrc, P, W, stream));
+    TRY(B200Q_PROF_GEMM, 2.0 * P * 2.0 * F * W,
+        b200q_linear_grouped(sorted ? y->esrc : y->h2, W, sorted ? nullptr : y->perm_tok, l.experts_gate_up, 2LL * F * W,
+                             y->egu, 2 * F, y->group_off, N, P, 2 * F, W, dt, y->tile_tab, y->n_tiles, stream));
+    TRY(EW, 3.0 * P * F * es, b200q_silu_glu(y->egu, y->eact, P, F, dt, stream));
+    TRY(B200Q_PROF_GEMM, 2.0 * P * (double)F * W,
+        b200q_linear_grouped(y->eact, F, nullptr, l.experts_down, (long long)W * F, y->eout, W, y->group_off, N, P, W, F, dt,
+                             y->tile_tab, y->n_tiles, stream));
+    if (d.shared_dim > 0 && !stacked) {
+      const int FS = d.shared_dim;
+      LIN(y->h2, W, l.shared_gate_up, nullptr, y->ffh, 2 * FS, 2 * FS, W, 0);
+      TRY(EW, 3.0 * T * FS * es, b200q_silu_glu(y->ffh, y->ffa, T, FS, dt, stream));
+      LIN(y->ffa, FS, l.shared_down, nullptr, y->shout, W, W, FS, 0);
+    }
+    return B200Q_OK;
+  };
+
+  // the embedding output, where a later pass adds it (a first layer that opens a pass keeps it itself)
   bool keep_x0 = false;
-  for (const auto& l : y->layers) keep_x0 = keep_x0 || l.d.inject;
-  if (keep_x0) TRY(EW, 8.0 * T * W, b200q_copy_f32(y->x, y->x0, (int64_t)T * W, stream));
+  for (const auto& l : y->layers) keep_x0 = keep_x0 || l.d.inject == B200Q_INJECT_MATRIX || l.d.inject == B200Q_INJECT_STEP_EMBED;
+  const bool kept_by_pass = keep_x0 && y->layers[0].d.inject == B200Q_INJECT_STEP;
+  if (lean)
+    for (const auto& l : y->layers)
+      if (l.rot_table && !l.rot_shared)
+        TRY(EW, 8.0 * T * l.d.rot_dims / 2,
+            b200q_rot_table(l.freq, l.mag, b->positions, T, l.d.rot_dims / 2, y->rot + l.rot_off * (int64_t)c.max_tokens, stream));
+  if (keep_x0 && !kept_by_pass) TRY(EW, 8.0 * T * W, b200q_copy_f32(y->x, y->x0, (int64_t)T * W, stream));
 
   int rot_layer = -1;  // the layer whose rotation y->rot holds
   for (int li = 0; li < c.n_layers; ++li) {
@@ -1139,12 +1318,53 @@ int layered_forward(b200q_model* m, const b200q_batch* b, void* stream) {
       // Every sum also writes what reads the new x next: the following norm's output, or x itself in the model dtype.
       const int NK = c.norm_kind, D = c.side_dim;
       const bool last = li + 1 == c.n_layers;
-      const int next_kind = last ? B200Q_NORM_NONE : NK;
-      const float* next_w = last ? nullptr : y->layers[li + 1].norm1;
-      if (li == 0)
+      // (a layer that opens a pass norms its x itself, after what comes ahead of the pass)
+      const bool open = !last && y->layers[li + 1].d.inject == B200Q_INJECT_NONE;
+      const int next_kind = open ? NK : B200Q_NORM_NONE;
+      const float* next_w = open ? y->layers[li + 1].norm1 : nullptr;
+      if (d.inject != B200Q_INJECT_NONE)
+        TRY(EW, (double)T * W * (8 + es),
+            b200q_pass_begin(y->x, d.inject == B200Q_INJECT_STEP_EMBED ? y->x0 : nullptr, l.step,
+                             li == 0 && kept_by_pass ? y->x0 : nullptr, l.norm1, y->h1, T, W, c.rms_eps, dt, stream));
+      else if (li == 0)
         TRY(EW, (double)T * W * (4 + es), b200q_row_norm(y->x, nullptr, NK, l.norm1, y->h1, T, W, c.rms_eps, dt, stream));
-      if ((rc = run_mixer(l))) return rc;
       const float* o_b = d.mixer == B200Q_MIXER_WINDOW_ATTN && d.proj_bias ? l.o_b : nullptr;
+      fold = lean && !o_b && d.ff != B200Q_FF_GEGLU;
+      if ((rc = run_mixer(l))) return rc;
+      if (fold) {
+        // RMS norms only: x <- x + n1b(mixer), x <- x + n2b(ff), the sums reading partial products or routed experts
+        TRY(EW, (double)T * W * (8 + 2 * es),
+            b200q_sandwich_close(y->x, splits > 1 ? (const void*)parts : y->mix, splits > 1 ? 1 : 0, splits, nullptr, nullptr, 0,
+                                 nullptr, l.norm1b, has_ff ? l.norm2 : next_w, has_ff ? y->h2 : y->h1, T, W, c.rms_eps, dt,
+                                 stream));
+        if (d.ff == B200Q_FF_CLAMPED) {
+          const int F = d.ff_dim;
+          // (steps of few tokens keep the plain product, as below)
+          if (l.gate_up_il && dt == B200Q_DTYPE_BF16 && W % 64 == 0 && T >= 512 &&
+              ((reinterpret_cast<uintptr_t>(y->h2) | reinterpret_cast<uintptr_t>(l.gate_up) |
+                reinterpret_cast<uintptr_t>(y->ffa)) & 15) == 0) {
+            TRY(B200Q_PROF_GEMM, 2.0 * T * 2.0 * F * W,
+                b200q_gemm_clamped_glu_bf16(y->h2, l.gate_up, nullptr, y->ffa, F, T, 2 * F, W, d.ff_limit, stream));
+          } else {
+            LIN(y->h2, W, l.gate_up, nullptr, y->ffh, 2 * F, 2 * F, W, 0);
+            TRY(EW, 3.0 * T * F * es,
+                b200q_clamped_glu_ex(y->ffh, 2 * F, nullptr, y->ffa, F, T, F, l.gate_up_il ? 128 : 0, d.ff_limit, dt, stream));
+          }
+          if ((rc = product(y->ffa, l.ff_down, y->ffo, F))) return rc;
+          TRY(EW, (double)T * W * (8 + 2 * es),
+              b200q_sandwich_close(y->x, splits > 1 ? (const void*)parts : y->ffo, splits > 1 ? 1 : 0, splits, nullptr, nullptr,
+                                   0, nullptr, l.norm2b, next_w, y->h1, T, W, c.rms_eps, dt, stream));
+        } else if (d.ff == B200Q_FF_MOE_GATED) {
+          if ((rc = run_moe_gated(l))) return rc;
+          const bool stacked = shared_stacked(d);
+          const int K = d.top_k + (stacked ? 1 : 0);
+          TRY(EW, (double)T * W * (8 + (1 + K) * es),
+              b200q_sandwich_close(y->x, y->eout, 0, 1, y->pair_pos, y->wts, K, d.shared_dim > 0 && !stacked ? y->shout : nullptr,
+                                   l.norm2b, next_w, y->h1, T, W, c.rms_eps, dt, stream));
+        }
+        if (y->tap) TRY(EW, 8.0 * T * W, b200q_copy_f32(y->x, y->tap + (int64_t)li * T * W, (int64_t)T * W, stream));
+        continue;
+      }
       const int after_kind = D > 0 ? B200Q_NORM_CAST : next_kind;  // what follows the layer's last sublayer
       const float* after_w = D > 0 ? nullptr : next_w;
       if (has_ff) {
@@ -1208,8 +1428,7 @@ int layered_forward(b200q_model* m, const b200q_batch* b, void* stream) {
                                  l.gate_up_il ? 128 : 0, d.ff_limit, dt, stream));
       // cosines and sines once per step for all layers of equal rotation
       const b200q_layer_desc* td = rot_layer < 0 ? nullptr : &y->layers[rot_layer].d;
-      if (d.rot_dims > 0 && !(td && td->rot_dims == d.rot_dims && td->rot_base == d.rot_base && td->rot_factor == d.rot_factor &&
-                              td->rot_original == d.rot_original && td->rot_fast == d.rot_fast && td->rot_slow == d.rot_slow)) {
+      if (d.rot_dims > 0 && !(td && same_rotation(*td, d))) {
         TRY(EW, 8.0 * T * d.rot_dims / 2, b200q_rot_table(l.freq, l.mag, b->positions, T, d.rot_dims / 2, y->rot, stream));
         rot_layer = li;
       }

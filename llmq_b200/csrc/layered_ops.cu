@@ -287,6 +287,44 @@ __global__ void __launch_bounds__(128) rope_q_kernel(const T* __restrict__ q, in
   }
 }
 
+// steps 1 and 2 in one for full-rank queries (CTA per token): proj = [q (heads x [dim | rot_dim]) | latent | shared
+// rotated key part].  Pairs (i, i + rot_dims/2) of the first rot_dims entries turn by the step's table.
+template <typename T>
+__global__ void __launch_bounds__(128) latent_prep_tab_kernel(const T* __restrict__ proj, int ldp, int heads, int dim,
+                                                              int kv_rank, int rot_dim, int rot_dims,
+                                                              const float2* __restrict__ table,
+                                                              const int32_t* __restrict__ slot_mapping,
+                                                              const float* __restrict__ w_kvn, float* __restrict__ qa,
+                                                              T* __restrict__ cache, float eps) {
+  extern __shared__ float2 turn_cs[];  // [rot_dims/2] (cos, sin)
+  __shared__ float red[32];
+  const int t = blockIdx.x, half = rot_dims / 2, QD = dim + rot_dim, RP = kv_rank + rot_dim;
+  for (int i = threadIdx.x; i < half; i += blockDim.x) turn_cs[i] = table[(long long)t * half + i];
+  const T* pr = proj + (long long)t * ldp;
+  const T* pc = pr + heads * QD;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < kv_rank; c += blockDim.x) {
+    const float v = ldf(pc + c);
+    ss = fmaf(v, v, ss);
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)kv_rank + eps);  // (its barriers also publish the table row)
+  auto turned = [&](const T* v, int d) -> float {
+    if (d >= rot_dims) return ldf(v + d);
+    const int i = d < half ? d : d - half;
+    const float a = ldf(v + i), b = ldf(v + i + half);
+    return d < half ? a * turn_cs[i].x - b * turn_cs[i].y : b * turn_cs[i].x + a * turn_cs[i].y;
+  };
+  for (int e = threadIdx.x; e < heads * rot_dim; e += blockDim.x) {
+    const int h = e / rot_dim, d = e % rot_dim;
+    qa[((long long)t * heads + h) * RP + kv_rank + d] = turned(pr + h * QD + dim, d);
+  }
+  const int slot = slot_mapping[t];
+  if (slot < 0) return;
+  T* row = cache + (long long)slot * RP;
+  for (int c = threadIdx.x; c < kv_rank; c += blockDim.x) stf(row + c, ldf(pc + c) * inv * w_kvn[c]);
+  for (int d = threadIdx.x; d < rot_dim; d += blockDim.x) stf(row + kv_rank + d, turned(pc + kv_rank, d));
+}
+
 // ------------------------------------------------------------------------------------------------
 // step 3: attention in the latent space.  The query of head h is qa[t,h,:] = [W_uk[h]^T q_unrotated |
 // q_rotated] (kv_rank + rot_dim values), a cached row is [latent c | rotated key part], so the score is
@@ -305,7 +343,8 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const float* __restric
                                                           const int32_t* __restrict__ row_seq,
                                                           const int32_t* __restrict__ positions, int heads,
                                                           int kv_rank, int rot_dim, int block_size, int window,
-                                                          float scale, const T* __restrict__ gate, int ld_gate,
+                                                          float scale, const float* __restrict__ sink,
+                                                          const T* __restrict__ gate, int ld_gate,
                                                           T* __restrict__ out) {
   extern __shared__ float sm[];
   const int RP = kv_rank + rot_dim, KS = RP + 1;
@@ -323,6 +362,10 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const float* __restric
     qs[e] = hh < heads ? qa[((long long)t * heads + hh) * RP + e % RP] : 0.f;
   }
   float m = -INFINITY, l = 0.f;
+  if (sink && live) {  // a logit of the denominator without key and value
+    m = sink[h];
+    l = 1.f;
+  }
   float acc[LATENT_ACC];
 #pragma unroll
   for (int i = 0; i < LATENT_ACC; ++i) acc[i] = 0.f;
@@ -399,6 +442,7 @@ __global__ void __launch_bounds__(128) latent_attn_mma_kernel(const float* __res
                                                               const int32_t* __restrict__ row_seq,
                                                               const int32_t* __restrict__ positions, int heads, int R,
                                                               int P, int block_size, int window, float scale,
+                                                              const float* __restrict__ sink,
                                                               const bf16* __restrict__ gate, int ld_gate,
                                                               bf16* __restrict__ out) {
   extern __shared__ __align__(16) uint8_t smraw[];
@@ -455,6 +499,14 @@ __global__ void __launch_bounds__(128) latent_attn_mma_kernel(const float* __res
   const uint32_t pa_off = (uint32_t)(((lane & 15) * LATENT_PLD + (lane >> 4) * 8) * 2);
   const int ntw = R / 32, dim_w = warp * (R / 4);
   float m_[2] = {-INFINITY, -INFINITY}, l_[2] = {0.f, 0.f};
+  if (sink) {  // every thread holds its rows' whole sums, so the sink's 1 belongs to each of them
+#pragma unroll
+    for (int r = 0; r < 2; ++r)
+      if (h0 + g + 8 * r < heads) {
+        m_[r] = sink[h0 + g + 8 * r];
+        l_[r] = 1.f;
+      }
+  }
   float o[NTW][4];
 #pragma unroll
   for (int i = 0; i < NTW; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
@@ -590,6 +642,7 @@ __global__ void __launch_bounds__(128) latent_attn_mma2_kernel(const float* __re
                                                                const int32_t* __restrict__ row_seq,
                                                                const int32_t* __restrict__ positions, int heads, int R,
                                                                int P, int block_size, int window, float scale,
+                                                               const float* __restrict__ sink,
                                                                const bf16* __restrict__ gate, int ld_gate,
                                                                bf16* __restrict__ out) {
   extern __shared__ __align__(16) uint8_t smraw[];
@@ -650,6 +703,14 @@ __global__ void __launch_bounds__(128) latent_attn_mma2_kernel(const float* __re
   const uint32_t kq_off = (uint32_t)((((lane & 7) + 8 * (lane >> 4)) * LDS + warp * KS * 16 + 8 * ((lane >> 3) & 1)) * 2);
   const int ntw = R / 32, dim_w = warp * (R / 4);
   float m_[2] = {-INFINITY, -INFINITY}, l_[2] = {0.f, 0.f};
+  if (sink) {  // every thread holds its rows' whole sums, so the sink's 1 belongs to each of them
+#pragma unroll
+    for (int r = 0; r < 2; ++r)
+      if (h0 + g + 8 * r < heads) {
+        m_[r] = sink[h0 + g + 8 * r];
+        l_[r] = 1.f;
+      }
+  }
   float o[NTW][4];
 #pragma unroll
   for (int i = 0; i < NTW; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
@@ -1389,6 +1450,22 @@ int b200q_latent_prep_ex(const void* proj, int ldp, int q_rank, int kv_rank, int
   return B200Q_OK;
 }
 
+int b200q_latent_prep_tab(const void* proj, int ldp, int heads, int dim, int kv_rank, int rot_dim, int rot_dims,
+                          const float* table, const int32_t* slot_mapping, const float* w_kvn, float* qa, void* cache, int T_,
+                          float eps, int dtype, void* stream) {
+  B200Q_CHECK_ARG(proj && slot_mapping && w_kvn && qa && cache && heads > 0 && dim >= 0 && kv_rank > 0 && rot_dim >= 0 &&
+                      rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= rot_dim && (rot_dims == 0 || table) &&
+                      ldp >= heads * (dim + rot_dim) + kv_rank + rot_dim && T_ >= 0 && eps >= 0.f && is_dtype(dtype),
+                  "latent_prep: bad argument (heads=%d dim=%d kv_rank=%d rot_dim=%d rot_dims=%d)", heads, dim, kv_rank, rot_dim,
+                  rot_dims);
+  if (T_ == 0) return B200Q_OK;
+  DISPATCH_T(dtype, (latent_prep_tab_kernel<T><<<T_, 128, (size_t)(rot_dims / 2 + 1) * sizeof(float2), as_stream(stream)>>>(
+                        (const T*)proj, ldp, heads, dim, kv_rank, rot_dim, rot_dims, (const float2*)table, slot_mapping, w_kvn,
+                        qa, (T*)cache, eps)));
+  B200Q_LAUNCH_CHECK();
+  return B200Q_OK;
+}
+
 int b200q_rope_pairs_q(const void* q, int heads, int dim, int rot_dim, int rot_dims, const double* freq,
                        const int32_t* positions, float* qa, int kv_rank, int T_, int dtype, void* stream) {
   return b200q_rope_pairs_q_ex(q, heads * (dim + rot_dim), heads, dim, rot_dim, rot_dims, freq, 1.f, positions, qa, kv_rank,
@@ -1420,6 +1497,14 @@ int b200q_latent_attn_ex(const float* qa, const void* cache, const int32_t* bloc
                          const int32_t* row_seq, const int32_t* positions, int T_, int heads, int kv_rank, int rot_dim,
                          int block_size, int window, float scale, const void* gate, int ld_gate, void* out, int dtype,
                          void* stream) {
+  return b200q_latent_attn_sink(qa, cache, block_table, bt_stride, row_seq, positions, T_, heads, kv_rank, rot_dim, block_size,
+                                window, scale, nullptr, gate, ld_gate, out, dtype, stream);
+}
+
+int b200q_latent_attn_sink(const float* qa, const void* cache, const int32_t* block_table, int bt_stride,
+                           const int32_t* row_seq, const int32_t* positions, int T_, int heads, int kv_rank, int rot_dim,
+                           int block_size, int window, float scale, const float* sink, const void* gate, int ld_gate,
+                           void* out, int dtype, void* stream) {
   B200Q_CHECK_ARG(!gate || ld_gate >= heads, "latent_attn: gate rows of stride %d hold fewer than %d heads", ld_gate, heads);
   B200Q_CHECK_ARG(qa && cache && block_table && row_seq && positions && out && heads > 0 && T_ >= 0 &&
                       block_size > 0 && window >= 0 && is_dtype(dtype),
@@ -1449,7 +1534,7 @@ int b200q_latent_attn_ex(const float* qa, const void* cache, const int32_t* bloc
                                     (int)sm3));                                                                   \
     latent_attn_mma2_kernel<NTW, KS><<<grid2, 128, sm3, as_stream(stream)>>>(                                      \
         qa, (const bf16*)cache, block_table, bt_stride, row_seq, positions, heads, kv_rank, rot_dim, block_size, \
-        window, scale, (const bf16*)gate, ld_gate, (bf16*)out);                                                   \
+        window, scale, sink, (const bf16*)gate, ld_gate, (bf16*)out);                                                   \
     B200Q_LAUNCH_CHECK();                                                                                         \
     return B200Q_OK;                                                                                              \
   } while (0)
@@ -1466,7 +1551,7 @@ int b200q_latent_attn_ex(const float* qa, const void* cache, const int32_t* bloc
                                     (int)sm2));                                                                   \
     latent_attn_mma_kernel<NTW><<<grid2, 128, sm2, as_stream(stream)>>>(                                          \
         qa, (const bf16*)cache, block_table, bt_stride, row_seq, positions, heads, kv_rank, rot_dim, block_size, \
-        window, scale, (const bf16*)gate, ld_gate, (bf16*)out);                                                   \
+        window, scale, sink, (const bf16*)gate, ld_gate, (bf16*)out);                                                   \
   } while (0)
       if (kv_rank <= 128) LATENT_MMA(4);
       else if (kv_rank <= 256) LATENT_MMA(8);
@@ -1483,7 +1568,7 @@ int b200q_latent_attn_ex(const float* qa, const void* cache, const int32_t* bloc
                                     (int)smem));                                                                   \
     latent_attn_kernel<TT, ACC><<<grid, 256, smem, as_stream(stream)>>>(                                           \
         qa, (const TT*)cache, block_table, bt_stride, row_seq, positions, heads, kv_rank, rot_dim, block_size,    \
-        window, scale, (const TT*)gate, ld_gate, (TT*)out);                                                        \
+        window, scale, sink, (const TT*)gate, ld_gate, (TT*)out);                                                        \
   } while (0)
 #define LATENT_BY_RANK(TT)                          \
   do {                                              \

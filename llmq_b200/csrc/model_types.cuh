@@ -47,6 +47,10 @@ struct b200q_layered_layer {
   // parallel form with a shared norm: fused projections of both sublayers, their biases, differential attention's factor
   const void *in = nullptr, *out = nullptr;
   const float *in_b = nullptr, *out_b = nullptr, *map_lambda = nullptr;
+  // softmax sink per head; the vector a pass begins with; the layer's place among the step's rotation tables (floats per token)
+  const float *sink = nullptr, *step = nullptr;
+  bool rot_table = false, rot_shared = false;
+  int64_t rot_off = 0;
   float mag = 1.f;  // factor of sine and cosine (YaRN)
   bool gate_up_il = false;  // gate_up rows interleaved in blocks of 128 (the fused product + gated unit's layout)
   std::vector<b200q_layered_layer> side;  // the mixer beside the first one (none or one)
@@ -61,6 +65,7 @@ struct b200q_layered {
   std::vector<b200q_layered_layer> layers;
   int64_t kv_block_bytes = 0;
   int64_t state_slot_floats = 0;
+  int64_t rot_floats = 0;  // floats per token of the step's rotation tables
   float* state = nullptr;
   int64_t n_slots = 0;
   float* tap = nullptr;

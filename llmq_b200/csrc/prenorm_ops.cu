@@ -205,30 +205,38 @@ __global__ void __launch_bounds__(256) decay_from_logits_kernel(float* __restric
 // correction and is masked to the kept groups (a masked expert counts as minus infinity, so negative choice
 // scores still beat it).  Ties go to the lowest index, for groups and for experts.
 // ------------------------------------------------------------------------------------------------
+// GATED: scores are the sigmoids of the logits, a group counts with the sum of its two largest choices, the weights are the
+// chosen scores as they are, and `shared` appends one pair per token for expert E with weight 1.
 constexpr int ROUTE_MAX_GROUPS = 256;
+template <bool GATED>
 __global__ void __launch_bounds__(128) moe_route_grouped_kernel(const float* __restrict__ logits,
                                                                 const float* __restrict__ corr, int Tn, int E, int top,
-                                                                int n_groups, int keep, int32_t* __restrict__ idx,
-                                                                float* __restrict__ wts) {
+                                                                int n_groups, int keep, int shared,
+                                                                int32_t* __restrict__ idx, float* __restrict__ wts) {
   __shared__ float gscore[4][ROUTE_MAX_GROUPS];
   const int wi = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * 4 + wi;
   if (t >= Tn) return;
   const float* z = logits + (long long)t * E;
-  float mx = -INFINITY;
-  for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
-  mx = warp_max(mx);
-  float sum = 0.f;
-  for (int e = lane; e < E; e += 32) sum += expf(z[e] - mx);
-  sum = warp_sum(sum);
-  const float inv = 1.f / sum;
-  auto score = [&](int e) { return expf(z[e] - mx) * inv; };
+  float mx = -INFINITY, inv = 1.f;
+  if (!GATED) {
+    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
+    mx = warp_max(mx);
+    float sum = 0.f;
+    for (int e = lane; e < E; e += 32) sum += expf(z[e] - mx);
+    inv = 1.f / warp_sum(sum);
+  }
+  auto score = [&](int e) { return GATED ? sigmoidf_(z[e]) : expf(z[e] - mx) * inv; };
   const int gs = E / n_groups;
   float* gsc = gscore[wi];
   for (int g = lane; g < n_groups; g += 32) {
-    float b = -INFINITY;
-    for (int e = g * gs; e < (g + 1) * gs; ++e) b = fmaxf(b, score(e) + corr[e]);
-    gsc[g] = b;
+    float b = -INFINITY, second = -INFINITY;
+    for (int e = g * gs; e < (g + 1) * gs; ++e) {
+      const float v = score(e) + corr[e];
+      second = fmaxf(second, fminf(b, v));
+      b = fmaxf(b, v);
+    }
+    gsc[g] = GATED && gs > 1 ? b + second : b;
   }
   __syncwarp();
   // a group is kept if fewer than `keep` groups rank before it (larger score, or equal score and lower index);
@@ -281,10 +289,15 @@ __global__ void __launch_bounds__(128) moe_route_grouped_kernel(const float* __r
     prev_v = bv;
     prev_i = bi;
   }
-  const float tot = warp_sum(lane < top ? chosen_s : 0.f);
+  const float tot = GATED ? 0.f : warp_sum(lane < top ? chosen_s : 0.f);
+  const int per = top + shared;
   if (lane < top) {
-    idx[(long long)t * top + lane] = chosen_i;
-    wts[(long long)t * top + lane] = chosen_s / (tot + 1e-20f);
+    idx[(long long)t * per + lane] = chosen_i;
+    wts[(long long)t * per + lane] = GATED ? chosen_s : chosen_s / (tot + 1e-20f);
+  }
+  if (shared && lane == 0) {
+    idx[(long long)t * per + top] = E;
+    wts[(long long)t * per + top] = 1.f;
   }
 }
 
@@ -509,11 +522,31 @@ int b200q_moe_route_grouped(const float* logits, const float* correction, int T_
                   "moe_route_grouped: bad argument (E=%d top=%d groups=%d keep=%d; groups divide E, at most %d groups, "
                   "top fits the kept groups)", E, top, n_groups, keep, ROUTE_MAX_GROUPS);
   if (T_ == 0) return B200Q_OK;
-  moe_route_grouped_kernel<<<(T_ + 3) / 4, 128, 0, as_stream(stream)>>>(logits, correction, T_, E, top, n_groups, keep, idx,
-                                                                       wts);
+  moe_route_grouped_kernel<false><<<(T_ + 3) / 4, 128, 0, as_stream(stream)>>>(logits, correction, T_, E, top, n_groups, keep,
+                                                                              0, idx, wts);
   B200Q_LAUNCH_CHECK();
   moe_plan_part_kernel<<<1, 1024, (size_t)(3 * E + 1) * sizeof(int32_t), as_stream(stream)>>>(
       idx, T_ * top, top, E, e_gemm, group_off, perm_tok, pair_pos, tile_tab, n_tiles);
+  B200Q_LAUNCH_CHECK();
+  return B200Q_OK;
+}
+
+int b200q_moe_route_gated(const float* logits, const float* correction, int T_, int E, int top, int n_groups, int keep,
+                          int shared, int32_t* idx, float* wts, int32_t* group_off, int32_t* perm_tok, int32_t* pair_pos,
+                          int32_t* tile_tab, int32_t* n_tiles, void* stream) {
+  B200Q_CHECK_ARG(!tile_tab == !n_tiles, "moe_route_gated: tile_tab and n_tiles go together");
+  B200Q_CHECK_ARG(logits && correction && idx && wts && group_off && perm_tok && pair_pos && T_ >= 0 && E > 0 && E + shared < 4096 &&
+                      top > 0 && top <= 32 && n_groups > 0 && n_groups <= ROUTE_MAX_GROUPS && E % n_groups == 0 && keep > 0 &&
+                      keep <= n_groups && top <= keep * (E / n_groups) && (shared == 0 || shared == 1),
+                  "moe_route_gated: bad argument (E=%d top=%d groups=%d keep=%d; groups divide E, at most %d groups, top fits "
+                  "the kept groups)", E, top, n_groups, keep, ROUTE_MAX_GROUPS);
+  if (T_ == 0) return B200Q_OK;
+  const int per = top + shared, n = E + shared;
+  moe_route_grouped_kernel<true><<<(T_ + 3) / 4, 128, 0, as_stream(stream)>>>(logits, correction, T_, E, top, n_groups, keep,
+                                                                             shared, idx, wts);
+  B200Q_LAUNCH_CHECK();
+  moe_plan_part_kernel<<<1, 1024, (size_t)(3 * n + 1) * sizeof(int32_t), as_stream(stream)>>>(
+      idx, T_ * per, per, n, n, group_off, perm_tok, pair_pos, tile_tab, n_tiles);
   B200Q_LAUNCH_CHECK();
   return B200Q_OK;
 }

@@ -3,6 +3,8 @@
 //
 //   row_norm:        y = norm(x[rows])                       dynamic tanh, RMS, or a plain cast
 //   sandwich_add:    x += mult * post(y + bias);  out = next(x)     one pass over the row, x stays fp32
+//   sandwich_close:  the same for RMS norms on both sides, y a plain row, split-K partial sums or a routed sum of experts
+//   pass_begin:      x += step (+ x0);  out = rms(x) * w             opens a pass over repeated layers
 //   gelu_glu:        y = gelu_tanh(g) * u
 //   token_side_gate: out = gelu_tanh(g) * table[token, col0 ..]
 //
@@ -137,6 +139,148 @@ __global__ void __launch_bounds__(256) sandwich_add_kernel(float* __restrict__ x
   }
 }
 
+// Where a closing sum finds y: `splits` partial rows (fp32 or model dtype) `split_stride` apart, or the chosen experts' rows
+// with their weights; y2: rows added on top.
+struct CloseSource {
+  const void* y;
+  const int32_t* pair_pos;
+  const float* wts;
+  const void* y2;
+  long long split_stride;
+  int splits, top;
+};
+template <typename TY, typename T, int V>
+__device__ __forceinline__ void close_value(const CloseSource& s, long long t, int W, int c, float (&a)[4]) {
+  const TY* y = (const TY*)s.y;
+  float b[4];
+  if (s.pair_pos) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) a[i] = 0.f;
+    for (int k = 0; k < s.top; ++k) {
+      const long long p = t * s.top + k;
+      const TY* r = y + (long long)s.pair_pos[p] * W + c;
+      const float w = s.wts[p];
+      if (V == 4) ld4(r, b);
+      else b[0] = ldf(r);
+#pragma unroll
+      for (int i = 0; i < V; ++i) a[i] = fmaf(w, b[i], a[i]);
+    }
+  } else {
+    const TY* r = y + t * W + c;
+    if (V == 4) ld4(r, a);
+    else a[0] = ldf(r);
+    for (int k = 1; k < s.splits; ++k) {
+      r += s.split_stride;
+      if (V == 4) ld4(r, b);
+      else b[0] = ldf(r);
+#pragma unroll
+      for (int i = 0; i < V; ++i) a[i] += b[i];
+    }
+  }
+  if (s.y2) {
+    const T* r = (const T*)s.y2 + t * W + c;
+    if (V == 4) ld4(r, b);
+    else b[0] = ldf(r);
+#pragma unroll
+    for (int i = 0; i < V; ++i) a[i] += b[i];
+  }
+}
+
+// CTA per row; rows of up to 256 * V * CLOSE_ROWS values stay in registers between y's norm, the sum and x's norm, the
+// rest of a longer row is worked out again
+constexpr int CLOSE_ROWS = 4;
+template <typename TY, typename T, int V>
+__global__ void __launch_bounds__(256) sandwich_close_kernel(float* __restrict__ x, CloseSource s,
+                                                             const float* __restrict__ post_w,
+                                                             const float* __restrict__ next_w, T* __restrict__ out, int W,
+                                                             float eps) {
+  __shared__ float red[32];
+  const long long t = blockIdx.x;
+  float* xr = x + t * W;
+  float v[CLOSE_ROWS][4];
+  float ss = 0.f;
+  auto sq = [&](const float (&a)[4]) {
+#pragma unroll
+    for (int i = 0; i < V; ++i) ss = fmaf(a[i], a[i], ss);
+  };
+  const int step = 256 * V, c0 = threadIdx.x * V;
+#pragma unroll
+  for (int q = 0; q < CLOSE_ROWS; ++q)
+    if (c0 + q * step < W) {
+      close_value<TY, T, V>(s, t, W, c0 + q * step, v[q]);
+      sq(v[q]);
+    }
+  for (int c = c0 + CLOSE_ROWS * step; c < W; c += step) {
+    float a[4];
+    close_value<TY, T, V>(s, t, W, c, a);
+    sq(a);
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)W + eps);
+  ss = 0.f;
+  auto add = [&](int c, float (&a)[4]) {  // a: y's value, then x's new one
+    float xv[4], w[4];
+    if (V == 4) {
+      ld4(xr + c, xv);
+      ld4(post_w + c, w);
+    } else {
+      xv[0] = xr[c];
+      w[0] = post_w[c];
+    }
+#pragma unroll
+    for (int i = 0; i < V; ++i) a[i] = fmaf(a[i] * inv, w[i], xv[i]);
+    if (V == 4) st4(xr + c, a);
+    else xr[c] = a[0];
+    sq(a);
+  };
+#pragma unroll
+  for (int q = 0; q < CLOSE_ROWS; ++q)
+    if (c0 + q * step < W) add(c0 + q * step, v[q]);
+  for (int c = c0 + CLOSE_ROWS * step; c < W; c += step) {
+    float a[4];
+    close_value<TY, T, V>(s, t, W, c, a);
+    add(c, a);
+  }
+  if (!next_w) return;
+  const float inv2 = 1.f / sqrtf(block_sum(ss, red) / (float)W + eps);
+  T* outr = out + t * W;
+  auto next = [&](int c, float (&a)[4]) {
+    float w[4];
+    if (V == 4) ld4(next_w + c, w);
+    else w[0] = next_w[c];
+#pragma unroll
+    for (int i = 0; i < V; ++i) a[i] = a[i] * inv2 * w[i];
+    if (V == 4) st4(outr + c, a);
+    else stf(outr + c, a[0]);
+  };
+#pragma unroll
+  for (int q = 0; q < CLOSE_ROWS; ++q)
+    if (c0 + q * step < W) next(c0 + q * step, v[q]);
+  for (int c = c0 + CLOSE_ROWS * step; c < W; c += step) {
+    float a[4];
+    if (V == 4) ld4(xr + c, a);
+    else a[0] = xr[c];
+    next(c, a);
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) pass_begin_kernel(float* __restrict__ x, const float* __restrict__ x0,
+                                                         const float* __restrict__ step, float* __restrict__ keep,
+                                                         const float* __restrict__ w, T* __restrict__ out, int W, float eps) {
+  __shared__ float red[32];
+  const long long base = (long long)blockIdx.x * W;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < W; c += blockDim.x) {
+    const float was = x[base + c];
+    if (keep) keep[base + c] = was;
+    const float v = (x0 ? was + x0[base + c] : was) + step[c];
+    x[base + c] = v;
+    ss = fmaf(v, v, ss);
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)W + eps);
+  for (int c = threadIdx.x; c < W; c += blockDim.x) stf(out + base + c, x[base + c] * inv * w[c]);  // each thread its own
+}
+
 // where column c's gate and up values lie in a [2F] row: block 0 = [g (F) | u (F)]; block b > 0 = gate and up
 // interleaved in blocks of b columns ([g b | u b | g b | u b ...])
 __device__ __forceinline__ void glu_columns(int c, int F, int block, int& g_at, int& u_at) {
@@ -268,6 +412,43 @@ int b200q_sandwich_add(float* x, const void* y, const float* bias, int post_kind
   else
     DISPATCH_T(dtype, (sandwich_add_kernel<T, 1><<<T_, 256, 0, as_stream(stream)>>>(
                           x, (const T*)y, bias, post_kind, post_w, mult, next_kind, next_w, (T*)out, W, eps)));
+  B200Q_LAUNCH_CHECK();
+  return B200Q_OK;
+}
+
+int b200q_sandwich_close(float* x, const void* y, int y_f32, int splits, const int32_t* pair_pos, const float* wts, int top,
+                         const void* y2, const float* post_w, const float* next_w, void* out, int T_, int W, float eps,
+                         int dtype, void* stream) {
+  B200Q_CHECK_ARG(x && y && post_w && T_ >= 0 && W > 0 && is_dtype(dtype) && eps >= 0.f && splits >= 1 &&
+                      (splits == 1 || y_f32 || dtype == B200Q_DTYPE_F32) && (!next_w || out),
+                  "sandwich_close: bad argument (W=%d splits=%d)", W, splits);
+  B200Q_CHECK_ARG(!pair_pos || (wts && top > 0 && splits == 1 && !y_f32), "sandwich_close: bad routed sum (top=%d)", top);
+  if (T_ == 0) return B200Q_OK;
+  const CloseSource s{y, pair_pos, wts, y2, (long long)T_ * W, splits, top};
+  const bool v4 = W % 4 == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(y) |
+                                  reinterpret_cast<uintptr_t>(y2) | reinterpret_cast<uintptr_t>(post_w) |
+                                  reinterpret_cast<uintptr_t>(next_w) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+  cudaStream_t st = as_stream(stream);
+#define CLOSE(TY, V)                                                                                                      \
+  DISPATCH_T(dtype, (sandwich_close_kernel<TY, T, V><<<T_, 256, 0, st>>>(x, s, post_w, next_w, (T*)out, W, eps)))
+  if (y_f32) {
+    if (v4) CLOSE(float, 4);
+    else CLOSE(float, 1);
+  } else {
+    if (v4) CLOSE(T, 4);
+    else CLOSE(T, 1);
+  }
+#undef CLOSE
+  B200Q_LAUNCH_CHECK();
+  return B200Q_OK;
+}
+
+int b200q_pass_begin(float* x, const float* x0, const float* step, float* keep, const float* w, void* out, int T_, int W,
+                     float eps, int dtype, void* stream) {
+  B200Q_CHECK_ARG(x && step && w && out && T_ >= 0 && W > 0 && eps >= 0.f && is_dtype(dtype) && (!keep || keep != x0),
+                  "pass_begin: bad argument (W=%d)", W);
+  if (T_ == 0) return B200Q_OK;
+  DISPATCH_T(dtype, (pass_begin_kernel<T><<<T_, 256, 0, as_stream(stream)>>>(x, x0, step, keep, w, (T*)out, W, eps)));
   B200Q_LAUNCH_CHECK();
   return B200Q_OK;
 }

@@ -5,7 +5,9 @@
 // fp32 query; ordinary softmax over the keys max(0, p - window + 1) .. p; one sigmoid gate number per head.
 // Options that other designs use: the first `keep_first` keys of a sequence stay visible behind the window (they are
 // visited first, as tiles of their own, then the window's keys), and scores may be soft-capped
-// (cap * tanh(score / cap)) before the softmax.
+// (cap * tanh(score / cap)) before the softmax; the denominator may hold a sink per head (a logit without key and value:
+// the softmax state starts from (sink, 1) instead of nothing); the gate may be a value per output channel; the
+// preparation may read the step's table of cosines and sines instead of working them out per token.
 // A scalar kernel (fp32 model, any head size) and tensor-core kernels for bf16 caches.  Scores, softmax state
 // and accumulators are fp32 in all.
 #include <stdlib.h>
@@ -73,7 +75,8 @@ template <typename T>
 __global__ void __launch_bounds__(128) window_attn_prep_opt_kernel(
     const T* __restrict__ proj, int ldp, int q_off, int k_off, int v_off, const float* __restrict__ bias, int heads,
     int kv_heads, int dim, int vdim, int qk_norm, const float* __restrict__ w_qn, const float* __restrict__ w_kn,
-    float eps, int rot_dims, const double* __restrict__ freq, float mag, const int32_t* __restrict__ positions,
+    float eps, int rot_dims, const double* __restrict__ freq, float mag, const float2* __restrict__ table,
+    const int32_t* __restrict__ positions,
     const int32_t* __restrict__ slot_mapping, const float* __restrict__ temp, float scale, float temp_coef,
     int temp_every, float* __restrict__ qs, T* __restrict__ cache) {
   extern __shared__ float sh[];
@@ -82,12 +85,18 @@ __global__ void __launch_bounds__(128) window_attn_prep_opt_kernel(
   float* cs = sh;                 // [rot_dims/2] cos | [rot_dims/2] sin
   float* qv = sh + rot_dims;      // [heads*dim]
   float* kv = qv + HD;            // [kv_heads*dim]
-  const int pos = positions[t];
+  const int pos = positions ? positions[t] : 0;
   for (int i = threadIdx.x; i < half; i += blockDim.x) {
-    double sn, c;
-    sincos((double)pos * freq[i], &sn, &c);
-    cs[i] = (float)c * mag;
-    cs[half + i] = (float)sn * mag;
+    if (table) {
+      const float2 v = table[(long long)t * half + i];
+      cs[i] = v.x;
+      cs[half + i] = v.y;
+    } else {
+      double sn, c;
+      sincos((double)pos * freq[i], &sn, &c);
+      cs[i] = (float)c * mag;
+      cs[half + i] = (float)sn * mag;
+    }
   }
   const T* pr = proj + (long long)t * ldp;
   for (int e = threadIdx.x; e < HD; e += blockDim.x) qv[e] = ldf(pr + q_off + e) + (bias ? bias[q_off + e] : 0.f);
@@ -150,8 +159,9 @@ __global__ void __launch_bounds__(256) window_attn_kernel(const float* __restric
                                                           const int32_t* __restrict__ row_seq,
                                                           const int32_t* __restrict__ positions, int heads, int kv_heads,
                                                           int dim, int vdim, int block_size, int window,
-                                                          int keep_first, float softcap,
-                                                          const T* __restrict__ gate, int ld_gate, T* __restrict__ out) {
+                                                          int keep_first, float softcap, const float* __restrict__ sink,
+                                                          const T* __restrict__ gate, int ld_gate, int channel_gate,
+                                                          T* __restrict__ out) {
   extern __shared__ float sm[];
   const int KS = dim + 1, VS = vdim + 1;
   float* qsm = sm;              // [8][dim]
@@ -171,6 +181,10 @@ __global__ void __launch_bounds__(256) window_attn_kernel(const float* __restric
     qsm[e] = hh < rep ? qs[((long long)t * heads + g * rep + hh) * dim + e % dim] : 0.f;
   }
   float m = -INFINITY, l = 0.f;
+  if (sink && live) {
+    m = sink[h];
+    l = 1.f;
+  }
   float acc[ACC];
 #pragma unroll
   for (int i = 0; i < ACC; ++i) acc[i] = 0.f;
@@ -215,13 +229,14 @@ __global__ void __launch_bounds__(256) window_attn_kernel(const float* __restric
     m = m_new;
   }
   if (!live) return;
-  const float gv = gate ? sigmoidf_(ldf(gate + (long long)t * ld_gate + h)) : 1.f;
+  const float gv = gate && !channel_gate ? sigmoidf_(ldf(gate + (long long)t * ld_gate + h)) : 1.f;
   const float inv = gv / l;
   T* o = out + ((long long)t * heads + h) * vdim;
 #pragma unroll
   for (int i = 0; i < ACC; ++i) {
     const int d = lane + 32 * i;
-    if (d < vdim) stf(o + d, acc[i] * inv);
+    if (d < vdim)
+      stf(o + d, acc[i] * inv * (channel_gate ? sigmoidf_(ldf(gate + (long long)t * ld_gate + (long long)h * vdim + d)) : 1.f));
   }
 }
 
@@ -242,8 +257,10 @@ __global__ void __launch_bounds__(256) window_attn_mma_kernel(const float* __res
                                                               const int32_t* __restrict__ seq_desc, int heads,
                                                               int kv_heads, int block_size, int window,
                                                               int keep_first, float softcap,
+                                                              const float* __restrict__ sink,
                                                               const bf16* __restrict__ gate, int ld_gate,
-                                                              bf16* __restrict__ out, int skip_single) {
+                                                              int channel_gate, bf16* __restrict__ out,
+                                                              int skip_single) {
   constexpr int LDK = D + 8, LDV = DV + 8;  // padded rows (bf16 elements): ldmatrix rows fall on different banks
   extern __shared__ __align__(16) uint8_t smraw[];
   const int nw = blockDim.x >> 5;
@@ -308,6 +325,10 @@ __global__ void __launch_bounds__(256) window_attn_mma_kernel(const float* __res
     lo_row[r] = (window > 0 && i < nrows) ? max(0, p_row[r] - window + 1) : 0;
   }
   float m_[2] = {WATT_NEG, WATT_NEG}, l_[2] = {0.f, 0.f};
+  if (sink) {  // counted once per row: by the first of the four threads that share it
+    m_[0] = m_[1] = sink[h];
+    if (q4 == 0) l_[0] = l_[1] = 1.f;
+  }
   float o[DV / 8][4];
 #pragma unroll
   for (int i = 0; i < DV / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
@@ -402,13 +423,19 @@ __global__ void __launch_bounds__(256) window_attn_mma_kernel(const float* __res
     const int i = gq + 8 * r;
     if (i >= nrows) continue;
     const long long t = sq.row0 + r0 + i;
-    const float gv = gate ? sigmoidf_(__bfloat162float(gate[t * ld_gate + h])) : 1.f;
+    const float gv = gate && !channel_gate ? sigmoidf_(__bfloat162float(gate[t * ld_gate + h])) : 1.f;
     const float inv = gv / l_[r];
     bf16* orow = out + (t * heads + h) * DV;
+    const bf16* grow = channel_gate ? gate + t * ld_gate + (long long)h * DV : nullptr;
 #pragma unroll
     for (int nt = 0; nt < DV / 8; ++nt) {
       const int d = nt * 8 + 2 * q4;
-      *reinterpret_cast<uint32_t*>(orow + d) = pack_bf16x2(o[nt][2 * r] * inv, o[nt][2 * r + 1] * inv);
+      float g0 = 1.f, g1 = 1.f;
+      if (grow) {
+        g0 = sigmoidf_(__bfloat162float(grow[d]));
+        g1 = sigmoidf_(__bfloat162float(grow[d + 1]));
+      }
+      *reinterpret_cast<uint32_t*>(orow + d) = pack_bf16x2(o[nt][2 * r] * inv * g0, o[nt][2 * r + 1] * inv * g1);
     }
   }
 }
@@ -429,8 +456,9 @@ __global__ void __launch_bounds__(128) window_attn_decode_mma_kernel(const float
                                                                      int bt_stride, const int32_t* __restrict__ seq_desc,
                                                                      int heads, int kv_heads, int block_size, int window,
                                                                      int keep_first, float softcap,
+                                                                     const float* __restrict__ sink,
                                                                      const bf16* __restrict__ gate, int ld_gate,
-                                                                     bf16* __restrict__ out) {
+                                                                     int channel_gate, bf16* __restrict__ out) {
   constexpr int LDK = D + 8, LDV = DV + 8, MS = DV + 2;
   extern __shared__ __align__(16) uint8_t smraw[];
   bf16* qsm = reinterpret_cast<bf16*>(smraw);    // [16][LDK]
@@ -480,6 +508,14 @@ __global__ void __launch_bounds__(128) window_attn_decode_mma_kernel(const float
   const uint32_t kq_off = (uint32_t)((((lane & 7) + 8 * (lane >> 4)) * LDK + 8 * ((lane >> 3) & 1)) * 2);
   const bool row_on[2] = {gq < rep, gq + 8 < rep};
   float m_[2] = {WATT_NEG, WATT_NEG}, l_[2] = {0.f, 0.f};
+  if (sink && warp == 0) {  // counted once: by the first warp's state, there by the first of a row's four threads
+#pragma unroll
+    for (int r = 0; r < 2; ++r)
+      if (row_on[r]) {
+        m_[r] = sink[g * rep + gq + 8 * r];
+        l_[r] = q4 == 0 ? 1.f : 0.f;
+      }
+  }
   float o[DV / 8][4];
 #pragma unroll
   for (int i = 0; i < DV / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
@@ -597,7 +633,7 @@ __global__ void __launch_bounds__(128) window_attn_decode_mma_kernel(const float
       den = fmaf(src[DV + 1], f, den);
     }
     const int h = g * rep + r;
-    const float gv = gate ? sigmoidf_(__bfloat162float(gate[t * ld_gate + h])) : 1.f;
+    const float gv = gate ? sigmoidf_(__bfloat162float(gate[t * ld_gate + (channel_gate ? h * DV + d : h)])) : 1.f;
     out[(t * heads + h) * DV + d] = __float2bfloat16_rn(num / den * gv);
   }
 }
@@ -605,6 +641,36 @@ __global__ void __launch_bounds__(128) window_attn_decode_mma_kernel(const float
 }  // namespace b200q
 
 using namespace b200q;
+
+static int window_attn_prep_any(const void* proj, int ldp, int q_off, int k_off, int v_off, const float* bias, int heads,
+                                int kv_heads, int dim, int vdim, int qk_norm, const float* w_qn, const float* w_kn, float eps,
+                                int rot_dims, const double* freq, float mag, const float2* table, const int32_t* positions,
+                                const int32_t* slot_mapping, const float* temp, float scale, float temp_coef, int temp_every,
+                                float* qs, void* cache, int T_, int dtype, void* stream) {
+  const bool own = k_off >= 0;
+  B200Q_CHECK_ARG(proj && qs && heads > 0 && kv_heads > 0 && dim > 0 && vdim > 0 && q_off >= 0 &&
+                      ldp >= q_off + heads * dim && rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dim && T_ >= 0 &&
+                      is_dtype(dtype) && temp_every >= 0,
+                  "window_attn_prep: bad argument (heads=%d kv_heads=%d dim=%d vdim=%d rot_dims=%d even, <= dim)", heads,
+                  kv_heads, dim, vdim, rot_dims);
+  B200Q_CHECK_ARG(!own || (slot_mapping && cache && v_off >= 0 && ldp >= k_off + kv_heads * dim &&
+                           ldp >= v_off + kv_heads * vdim),
+                  "window_attn_prep: bad key / value columns (k_off=%d v_off=%d ldp=%d)", k_off, v_off, ldp);
+  B200Q_CHECK_ARG(qk_norm >= 0 && qk_norm <= 2 && (qk_norm == 0 || (w_qn && (!own || w_kn))) && eps >= 0.f,
+                  "window_attn_prep: bad query / key norm (%d)", qk_norm);
+  if (T_ == 0) return B200Q_OK;
+  const size_t smem = (size_t)(std::max(rot_dims, 1) + heads * dim + kv_heads * dim) * sizeof(float);
+  B200Q_CHECK_ARG(smem <= 200 * 1024, "window_attn_prep: heads * dim too large for one CTA");
+  DISPATCH_T(dtype, {
+    auto kern = window_attn_prep_opt_kernel<T>;
+    if (smem > 48 * 1024) B200Q_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    kern<<<T_, 128, smem, as_stream(stream)>>>((const T*)proj, ldp, q_off, k_off, v_off, bias, heads, kv_heads, dim, vdim,
+                                               qk_norm, w_qn, w_kn, eps, rot_dims, freq, mag, table, positions, slot_mapping,
+                                               temp, scale, temp_coef, temp_every, qs, (T*)cache);
+  });
+  B200Q_LAUNCH_CHECK();
+  return B200Q_OK;
+}
 
 extern "C" {
 
@@ -630,29 +696,20 @@ int b200q_window_attn_prep_ex(const void* proj, int ldp, int q_off, int k_off, i
                               int rot_dims, const double* freq, float mag, const int32_t* positions,
                               const int32_t* slot_mapping, const float* temp, float scale, float temp_coef, int temp_every,
                               float* qs, void* cache, int T_, int dtype, void* stream) {
-  const bool own = k_off >= 0;
-  B200Q_CHECK_ARG(proj && positions && qs && heads > 0 && kv_heads > 0 && dim > 0 && vdim > 0 && q_off >= 0 &&
-                      ldp >= q_off + heads * dim && rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dim &&
-                      (rot_dims == 0 || freq) && T_ >= 0 && is_dtype(dtype) && temp_every >= 0,
-                  "window_attn_prep: bad argument (heads=%d kv_heads=%d dim=%d vdim=%d rot_dims=%d even, <= dim)", heads,
-                  kv_heads, dim, vdim, rot_dims);
-  B200Q_CHECK_ARG(!own || (slot_mapping && cache && v_off >= 0 && ldp >= k_off + kv_heads * dim &&
-                           ldp >= v_off + kv_heads * vdim),
-                  "window_attn_prep: bad key / value columns (k_off=%d v_off=%d ldp=%d)", k_off, v_off, ldp);
-  B200Q_CHECK_ARG(qk_norm >= 0 && qk_norm <= 2 && (qk_norm == 0 || (w_qn && (!own || w_kn))) && eps >= 0.f,
-                  "window_attn_prep: bad query / key norm (%d)", qk_norm);
-  if (T_ == 0) return B200Q_OK;
-  const size_t smem = (size_t)(std::max(rot_dims, 1) + heads * dim + kv_heads * dim) * sizeof(float);
-  B200Q_CHECK_ARG(smem <= 200 * 1024, "window_attn_prep: heads * dim too large for one CTA");
-  DISPATCH_T(dtype, {
-    auto kern = window_attn_prep_opt_kernel<T>;
-    if (smem > 48 * 1024) B200Q_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    kern<<<T_, 128, smem, as_stream(stream)>>>((const T*)proj, ldp, q_off, k_off, v_off, bias, heads, kv_heads, dim, vdim,
-                                               qk_norm, w_qn, w_kn, eps, rot_dims, freq, mag, positions, slot_mapping,
-                                               temp, scale, temp_coef, temp_every, qs, (T*)cache);
-  });
-  B200Q_LAUNCH_CHECK();
-  return B200Q_OK;
+  B200Q_CHECK_ARG(positions && (rot_dims == 0 || freq), "window_attn_prep: positions or frequencies are missing");
+  return window_attn_prep_any(proj, ldp, q_off, k_off, v_off, bias, heads, kv_heads, dim, vdim, qk_norm, w_qn, w_kn, eps,
+                              rot_dims, freq, mag, nullptr, positions, slot_mapping, temp, scale, temp_coef, temp_every, qs,
+                              cache, T_, dtype, stream);
+}
+
+int b200q_window_attn_prep_tab(const void* proj, int ldp, int q_off, int k_off, int v_off, const float* bias, int heads,
+                               int kv_heads, int dim, int vdim, int qk_norm, const float* w_qn, const float* w_kn, float eps,
+                               int rot_dims, const float* table, const int32_t* slot_mapping, float scale, float* qs,
+                               void* cache, int T_, int dtype, void* stream) {
+  B200Q_CHECK_ARG(rot_dims == 0 || table, "window_attn_prep: the table is missing");
+  return window_attn_prep_any(proj, ldp, q_off, k_off, v_off, bias, heads, kv_heads, dim, vdim, qk_norm, w_qn, w_kn, eps,
+                              rot_dims, nullptr, 1.f, (const float2*)table, nullptr, slot_mapping, nullptr, scale, 0.f, 0, qs,
+                              cache, T_, dtype, stream);
 }
 
 static int window_attn_mma_mode() {  // B200Q_WINDOW_ATTN_MMA=0: the scalar kernel everywhere
@@ -686,6 +743,18 @@ int b200q_window_attn_ex(const float* qs, const void* cache, const int32_t* bloc
                          const int32_t* row_seq, const int32_t* positions, const int32_t* seq_desc, int n_seqs, int T_,
                          int heads, int kv_heads, int dim, int vdim, int block_size, int window, int keep_first,
                          float softcap, const void* gate, int ld_gate, void* out, int dtype, void* stream) {
+  return b200q_window_attn_sink(qs, cache, block_table, bt_stride, row_seq, positions, seq_desc, n_seqs, T_, heads, kv_heads,
+                                dim, vdim, block_size, window, keep_first, softcap, nullptr, gate, ld_gate, 0, out, dtype,
+                                stream);
+}
+
+int b200q_window_attn_sink(const float* qs, const void* cache, const int32_t* block_table, int bt_stride,
+                           const int32_t* row_seq, const int32_t* positions, const int32_t* seq_desc, int n_seqs, int T_,
+                           int heads, int kv_heads, int dim, int vdim, int block_size, int window, int keep_first,
+                           float softcap, const float* sink, const void* gate, int ld_gate, int channel_gate, void* out,
+                           int dtype, void* stream) {
+  B200Q_CHECK_ARG(!channel_gate || (gate && ld_gate >= heads * vdim), "window_attn: a gate per channel needs rows of %d values",
+                  heads * vdim);
   B200Q_CHECK_ARG(keep_first >= 0 && softcap >= 0.f, "window_attn: bad kept keys (%d) or soft cap (%g)", keep_first,
                   (double)softcap);
   if (window <= 0) keep_first = 0;  // every earlier key is visible anyway
@@ -725,8 +794,9 @@ int b200q_window_attn_ex(const float* qs, const void* cache, const int32_t* bloc
                                         (int)msm));                                                                      \
       window_attn_mma_kernel<DD, DDV, CC><<<mgrid, nw * 32, msm, st>>>(qs, (const bf16*)cache, block_table, bt_stride,       \
                                                                    seq_desc, heads, kv_heads, block_size, window,        \
-                                                                   keep_first, softcap,                                  \
-                                                                   (const bf16*)gate, ld_gate, (bf16*)out, dec ? 1 : 0); \
+                                                                   keep_first, softcap, sink,                            \
+                                                                   (const bf16*)gate, ld_gate, channel_gate, (bf16*)out, \
+                                                                   dec ? 1 : 0);                                         \
       B200Q_LAUNCH_CHECK();                                                                                              \
     }                                                                                                                    \
     if (dec) {                                                                                                           \
@@ -734,7 +804,8 @@ int b200q_window_attn_ex(const float* qs, const void* cache, const int32_t* bloc
       if (dsm > 48 * 1024)                                                                                               \
         B200Q_CUDA(cudaFuncSetAttribute(dk, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)dsm));                     \
       dk<<<dgrid, 128, dsm, st>>>(qs, (const bf16*)cache, block_table, bt_stride, seq_desc, heads, kv_heads, block_size, \
-                                  window, keep_first, softcap, (const bf16*)gate, ld_gate, (bf16*)out);                  \
+                                  window, keep_first, softcap, sink, (const bf16*)gate, ld_gate, channel_gate,           \
+                                  (bf16*)out);                                                                           \
       B200Q_LAUNCH_CHECK();                                                                                              \
     }                                                                                                                    \
   } while (0)
@@ -755,7 +826,8 @@ int b200q_window_attn_ex(const float* qs, const void* cache, const int32_t* bloc
       auto kern = window_attn_kernel<T, ACC>;                                                                             \
       if (smem > 48 * 1024) B200Q_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
       kern<<<grid, 256, smem, st>>>(qs, (const T*)cache, block_table, bt_stride, row_seq, positions, heads, kv_heads, dim, \
-                                    vdim, block_size, window, keep_first, softcap, (const T*)gate, ld_gate, (T*)out);      \
+                                    vdim, block_size, window, keep_first, softcap, sink, (const T*)gate, ld_gate,         \
+                                    channel_gate, (T*)out);                                                                \
     });                                                                                                                   \
   } while (0)
   if (vdim <= 64) SCALAR(2);

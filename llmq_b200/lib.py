@@ -73,6 +73,7 @@ ARCH_NORIDRA = 3
 ARCH_PALUZEN = 4
 ARCH_KABAVIK = 5
 ARCH_LIPEDRA = 6
+ARCH_FIMILORN = 7
 FORM_PARALLEL = 0
 FORM_POSTNORM = 1
 FORM_PRENORM = 2
@@ -92,6 +93,7 @@ MIXER_LIGHTNING = 6
 MIXER_WINDOW_ATTN = 7
 MIXER_DECAY_MIX = 8
 MIXER_DIFF_ATTN = 9
+MIXER_RETENTION = 10
 FF_NONE = 0
 FF_POLYNORM = 1
 FF_MOE = 2
@@ -100,6 +102,11 @@ FF_RELU2 = 4
 FF_MOE_GROUPED = 5
 FF_GEGLU = 6
 FF_CLAMPED = 7
+FF_MOE_GATED = 8
+INJECT_NONE = 0
+INJECT_MATRIX = 1
+INJECT_STEP = 2
+INJECT_STEP_EMBED = 3
 
 
 class LayerDesc(C.Structure):
@@ -118,6 +125,7 @@ class LayerDesc(C.Structure):
         ("head_gate", C.c_int32), ("q_temp_coef", C.c_float), ("q_temp_every", C.c_int32),
         ("rot_factor", C.c_double), ("rot_original", C.c_double), ("rot_fast", C.c_double), ("rot_slow", C.c_double),
         ("diff", C.c_float), ("ff_limit", C.c_float),
+        ("sink", C.c_int32), ("channel_gate", C.c_int32), ("rot_half", C.c_int32),
     ]
 
 
@@ -295,6 +303,18 @@ SIGNATURES = {
     "b200q_diff_attn": (_i, [_vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _f, _f, _vp, _i, _vp, _i, _i,
                              _vp]),
     "b200q_wait_failures": (_i, []),
+    # retention, softmax sinks, group-routed gated experts
+    "b200q_retention_scratch_floats": (_i64, [_i, _i, _i]),
+    "b200q_retention": (_i, [_vp, _i, _i, _i, _i, _i, _vp, _vp, _vp, _ll, _vp, _vp, _i, _i, _f, _vp, _vp, _i, _i, _vp]),
+    "b200q_window_attn_prep_tab": (_i, [_vp, _i, _i, _i, _i, _vp, _i, _i, _i, _i, _i, _vp, _vp, _f, _i, _vp, _vp, _f, _vp,
+                                        _vp, _i, _i, _vp]),
+    "b200q_window_attn_sink": (_i, [_vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _vp, _vp, _i,
+                                    _i, _vp, _i, _vp]),
+    "b200q_latent_prep_tab": (_i, [_vp, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _i, _f, _i, _vp]),
+    "b200q_latent_attn_sink": (_i, [_vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _vp, _vp, _i, _vp, _i, _vp]),
+    "b200q_moe_route_gated": (_i, [_vp, _vp, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp]),
+    "b200q_sandwich_close": (_i, [_vp, _vp, _i, _i, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _f, _i, _vp]),
+    "b200q_pass_begin": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _f, _i, _vp]),
     "b200q_model_create_layered": (_i, [C.POINTER(ModelConfig), C.POINTER(LayerDesc), C.POINTER(_vp)]),
     "b200q_model_kv_block_bytes": (_i64, [_vp]),
     "b200q_model_state_slot_bytes": (_i64, [_vp]),
