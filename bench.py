@@ -699,12 +699,12 @@ def run_compare(args):
             kind = getattr(ly, "kind", None)        # Paluzen's layer runs (a repeated layer counts once per pass)
             if hasattr(ly, "diff"):                 # Lipedra: two key maps and one value per key head, every earlier key
                 cache += B * (C0 + 1) * ly.kv_heads * (2 * ly.dim + ly.vdim) * 2
-            elif kind in ("attention", "attention_2") and hasattr(ly, "keep_first"):   # Kabavik: window + kept first keys
-                seen = min(C0 + 1, ly.window + ly.keep_first) if ly.window else C0 + 1
+            elif kind in ("attention", "attention_2"):   # Kabavik: window + kept first keys; Fimilorn: every earlier key
+                seen = min(C0 + 1, ly.window + getattr(ly, "keep_first", 0)) if ly.window else C0 + 1
                 cache += B * seen * ly.kv_heads * (ly.dim + ly.vdim) * 2
             elif kind == "latent_attention":
                 cache += B * min(C0 + 1, ly.window or C0 + 1) * (ly.kv_rank + ly.rot_dim) * 2
-            elif kind == "lightning":
+            elif kind in ("lightning", "retention"):
                 state += B * ly.heads * ly.dim * ly.vdim * 4 * 2
             elif kind == "parallel":
                 cache += B * min(C0 + 1, ly.window or C0 + 1) * ly.kv_heads * (ly.dim + ly.vdim) * 2
@@ -723,7 +723,7 @@ def run_compare(args):
 
     def prefill_attention_flops(spec):
         """score and value products of the cache-reading attention layers over the prefill workload (Lipedra's two maps,
-        Kabavik's three mixers, Paluzen's window attention)"""
+        Kabavik's three mixers, Paluzen's window attention, Fimilorn's two)"""
         fl = 0.0
         for ly in spec.layers:
             kind = getattr(ly, "kind", None)
@@ -731,7 +731,7 @@ def run_compare(args):
                 per_key = 2.0 * ly.heads * 2 * (ly.dim + ly.vdim)
             elif kind in ("attention", "attention_2", "parallel"):
                 per_key = 2.0 * ly.heads * (ly.dim + ly.vdim)
-            elif kind == "latent_attention" and hasattr(ly, "keep_first"):
+            elif kind == "latent_attention":
                 per_key = 2.0 * ly.heads * (2 * ly.kv_rank + ly.rot_dim)
             else:
                 continue
@@ -743,7 +743,7 @@ def run_compare(args):
     frac = lambda by, ms: round(by / (ms * 1e-3) / 1e9 / peaks["hbm_gbs"], 3) if ms > 0 else None
     tf = lambda fl, ms: round(fl / (ms * 1e-3) / 1e12 / peaks["bf16_tflops"], 3) if ms > 0 else None
     results = {}
-    if args.compare in ("noridra", "paluzen", "kabavik", "lipedra"):
+    if args.compare in ("noridra", "paluzen", "kabavik", "lipedra", "fimilorn"):
         # the design beside the closest existing one at equal width and layer count: Noridra beside Ramopel
         # (layered, recurrent state slots, routed experts); Paluzen beside Noridra (windowed / chunked grouped-query
         # attention on the tensor cores, decayed outer-product states, routed experts)
@@ -751,13 +751,15 @@ def run_compare(args):
         # norms, gated feed-forwards through the same GEMM)
         # Lipedra beside Kabavik (grouped-query attention with biases over a paged cache, gated feed-forwards with the
         # unit in the product's epilogue, borrowed keys and values)
-        new, old = args.compare, {"noridra": "ramopel", "paluzen": "noridra", "kabavik": "paluzen",
-                                  "lipedra": "kabavik"}[args.compare]
+        # Fimilorn beside Kabavik (sandwich norms, grouped-query and latent attention) and Paluzen (constant-decay states,
+        # group-routed experts)
+        new, olds = args.compare, {"noridra": ["ramopel"], "paluzen": ["noridra"], "kabavik": ["paluzen"],
+                                   "lipedra": ["kabavik"], "fimilorn": ["kabavik", "paluzen"]}[args.compare]
         for key in (args.compare_sizes or f"{new}-1b,{new}-3b").split(","):
-            nspec, rspec = BUILTIN_SPECS[key], BUILTIN_SPECS[key.replace(new, old)]
-            n, r = measure(nspec), measure(rspec)
+            arms = [(name, BUILTIN_SPECS[key.replace(new, name)]) for name in [new] + olds]
+            arms = [(name, spec, measure(spec)) for name, spec in arms]
             roof = {}
-            for name, spec, m in ((new, nspec, n), (old, rspec, r)):
+            for name, spec, m in arms:
                 cache, state = decode_bytes(spec)
                 k = m["decode"]["kernel_ms_per_step"]
                 pf = 2.0 * (spec.weight_bytes_per_token() / 2 - spec.vocab * spec.width) * n_p * S_p
@@ -768,9 +770,9 @@ def run_compare(args):
                               "prefill_attention_of_cublas": tf(prefill_attention_flops(spec),
                                                                 m["prefill"]["kernel_ms_per_run"]["decode_attn"]),
                               "decode_cache_mb": round(cache / 1e6, 2), "decode_state_mb": round(state / 1e6, 2)}
-            results[key] = {new: n, old + "_equal_size": r,
-                            "matrix_gb_per_token": {new: round(nspec.weight_bytes_per_token() / 1e9, 3),
-                                                    old: round(rspec.weight_bytes_per_token() / 1e9, 3)},
+            results[key] = {**{name if name == new else name + "_equal_size": m for name, _, m in arms},
+                            "matrix_gb_per_token": {name: round(spec.weight_bytes_per_token() / 1e9, 3)
+                                                    for name, spec, _ in arms},
                             "roofline": roof}
         print(json.dumps({"compare": new, "dtype": "bf16", "data": "synthetic (random weights, random ids)",
                           "peaks": peaks, "workload": {"prefill": f"{n_p} prompts x {S_p} tokens",
@@ -844,10 +846,10 @@ def main():
     ap.add_argument("--cpu-budget-s", type=float, default=10.0)
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--dry-run", action="store_true", help="host-logic self-test without a GPU (not a measurement)")
-    ap.add_argument("--compare", default=None, choices=["ramopel", "noridra", "paluzen", "kabavik", "lipedra"],
+    ap.add_argument("--compare", default=None, choices=["ramopel", "noridra", "paluzen", "kabavik", "lipedra", "fimilorn"],
                     help="instead of the headline workload: prefill / decode throughput of this design beside the closest "
                          "existing model of equal size (ramopel: a Llama decoder; noridra: Ramopel; paluzen: Noridra; kabavik: Paluzen; "
-                         "lipedra: Kabavik), random weights, one JSON line")
+                         "lipedra: Kabavik; fimilorn: Kabavik and Paluzen), random weights, one JSON line")
     ap.add_argument("--compare-sizes", default=None, help="builtin sizes, default <design>-1b,<design>-3b")
     ap.add_argument("--compare-prompt", type=int, default=2048)
     ap.add_argument("--compare-prompts", type=int, default=4)
