@@ -580,12 +580,13 @@ int b200q_window_attn_prep_tab(const void* proj_dev, int ldp, int q_off, int k_o
                                const int32_t* slot_mapping_dev, float scale, float* qs_dev, void* cache_dev, int T,
                                int dtype, void* stream);
 /* b200q_window_attn_ex with a softmax sink (fp32 [heads], NULL: none: the denominator also holds exp(sink[h])) and, with
- * channel_gate, a gate value per output channel (gate rows of heads*vdim values instead of heads) */
+ * channel_gate, a gate value per output channel (gate rows of heads*vdim values instead of heads).  max_portion as in
+ * b200q_diff_attn (grid sizes only). */
 int b200q_window_attn_sink(const float* qs_dev, const void* cache_dev, const int32_t* block_table_dev, int bt_stride,
                            const int32_t* row_seq_dev, const int32_t* positions_dev, const int32_t* seq_desc_dev,
                            int n_seqs, int T, int heads, int kv_heads, int dim, int vdim, int block_size, int window,
                            int keep_first, float softcap, const float* sink_dev, const void* gate_dev, int ld_gate,
-                           int channel_gate, void* out_dev, int dtype, void* stream);
+                           int channel_gate, int max_portion, void* out_dev, int dtype, void* stream);
 /* latent attention with full-rank queries, steps 1 and 2 in one: proj rows = [q (heads x [dim | rot_dim]) | latent
  * (kv_rank) | shared rotated key (rot_dim)];  cache row slot_mapping[t] = [latent / rms * w_kvn | turned key],
  * qa[t, h, kv_rank ..] = turned query part; pairs (i, i + rot_dims/2) of the first rot_dims, by `table` */
@@ -597,6 +598,23 @@ int b200q_latent_attn_sink(const float* qa_dev, const void* cache_dev, const int
                            const int32_t* row_seq_dev, const int32_t* positions_dev, int T, int heads, int kv_rank,
                            int rot_dim, int block_size, int window, float scale, const float* sink_dev,
                            const void* gate_dev, int ld_gate, void* out_dev, int dtype, void* stream);
+/* Latent attention of prompt portions over expanded keys and values (bf16; single tokens of the step are left alone, they
+ * read the latents themselves): b200q_latent_gather collects the latents that every portion of the step sees (positions
+ * max(0, pos0 - window + 1) .. pos0 + n - 1; window 0: from 0), sequence by sequence, into dense rows out [rows][kv_rank]
+ * (at most max_rows) and writes span[s] = {first row, first position} per sequence; the caller expands them to keys
+ * [rows][heads*dim] and values [rows][heads*vdim]; b200q_latent_portion_attn then reads queries as [unrotated | ...] rows q
+ * (stride ldq, head h at h * (dim + rot_dim)), their turned parts behind qa[t, h, kv_rank], the turned key parts from the
+ * cache, and writes out [T, heads*vdim].  longest_span / longest: most rows / tokens of any portion.
+ * b200q_latent_expand_ok says whether the sizes are taken. */
+int b200q_latent_expand_ok(int heads, int dim, int rot_dim, int vdim, int kv_rank, int block_size, int dtype);
+int b200q_latent_gather(const void* cache_dev, const int32_t* block_table_dev, int bt_stride, const int32_t* seq_desc_dev,
+                        int n_seqs, int longest_span, int window, int block_size, int kv_rank, int rot_dim, int max_rows,
+                        void* out_dev, int32_t* span_dev, void* stream);
+int b200q_latent_portion_attn(const void* q_dev, int ldq, const float* qa_dev, const void* keys_dev, const void* values_dev,
+                              const int32_t* span_dev, const void* cache_dev, const int32_t* block_table_dev, int bt_stride,
+                              const int32_t* seq_desc_dev, int n_seqs, int longest, int heads, int dim, int rot_dim, int vdim,
+                              int kv_rank, int block_size, int window, float scale, const float* sink_dev,
+                              const void* gate_dev, int ld_gate, void* out_dev, void* stream);
 /* routing of B200Q_FF_MOE_GATED over fp32 router logits [T, E]: s = sigmoid(logits), choice = s + correction; only experts
  * of the keep best of n_groups groups (score: sum of the two largest choices of the group) may be chosen; the top largest
  * choices (ties: lowest index) -> idx, wts = s.  shared 1: every token has one more pair, expert E with weight 1.  Outputs
@@ -888,6 +906,8 @@ typedef struct b200q_batch {
   const int32_t* row_seq;       /* [T]                                                           */
   int32_t no_sampling;          /* 1: stop after the logits (sample_rows may then hold up to max_logit_rows rows) */
   int32_t max_portion;          /* most tokens any sequence brings to this step; 0 = unknown     */
+  const int32_t* h_seq_desc;    /* host copy of seq_desc for the duration of the call, single-token sequences first;
+                                   NULL = unknown                                                */
 } b200q_batch;
 
 int b200q_model_create(const b200q_model_config* cfg, b200q_model_t* out);
@@ -932,7 +952,8 @@ int b200q_model_create(const b200q_model_config* cfg, b200q_model_t* out);
  *   window attention (bare, channel_gate, qk_norm 1, sink): "mix.proj" [roundup64(q + k + v + gate rows), W],
  *     "mix.q_norm" [1, heads*dim], "mix.k_norm" [1, kv_heads*dim], "mix.sink" [1, heads], "mix.o"
  *   latent attention (q_rank 0, sink): "mix.down" [roundup64(q rows + kv_rank + rot_dim), W], "mix.kv_norm", "mix.sink",
- *     "mix.uk_t", "mix.uv", "mix.o"
+ *     "mix.uk_t", "mix.uv", "mix.o", optionally "mix.uk" [heads*dim, kv_rank] (the key up-projection as it is: prompt
+ *     portions then read expanded keys and values where the sizes allow)
  *   clamped ff: "mlp.gate_up" or "mlp.gate_up_il" [2*ff, W], "mlp.down"
  *   gated experts: "mlp.router" [E, W], "mlp.router_bias" [1, E] (the correction), "mlp.experts_gate_up" [N*2*ff, W],
  *     "mlp.experts_down" [N*W, ff]; a shared expert as large as the others is expert E of these stacks (N = E + 1), one

@@ -752,6 +752,7 @@ static int launch_step(b200q_engine* e, InFlightStep& step, std::vector<Request*
     b.max_portion = 0;
     for (Request* r : sched) b.max_portion = std::max(b.max_portion, (int32_t)r->n_sched);
     b.seq_desc = e->d_meta + (sdesc - h_meta);
+    b.h_seq_desc = sdesc;
     b.row_seq = e->d_meta + (rseq - h_meta);
     b.no_sampling = replay ? 1 : 0;
     b.sum_ctx_dec = 0;

@@ -229,7 +229,7 @@ int check_layered(const b200q_model_config* c, const b200q_layer_desc* L) {
 // widest use of every workspace buffer over the layers
 struct Widths {
   int64_t proj = 1, cq = 1, q = 1, qa = 1, olat = 1, attn = 1, ffh = 1, ffa = 1, experts = 1, pairs = 1, egu = 1,
-          eact = 1, delta = 0, cvf = 0, baf = 0, dtr = 0, xc = 0, xp = 0, blend = 0, rot = 0;
+          eact = 1, delta = 0, cvf = 0, baf = 0, dtr = 0, xc = 0, xp = 0, blend = 0, rot = 0, lat = 0, lat_k = 0, lat_v = 0;
   bool moe = false, shared = false, hf = false, side = false, inject = false, keep_x0 = false;
 };
 int64_t pad64(int64_t v) { return (v + 63) & ~(int64_t)63; }
@@ -286,6 +286,11 @@ Widths widths_of(const b200q_model_config& c, const std::vector<b200q_layered_la
       if (d.q_rank > 0) w.q = std::max<int64_t>(w.q, (int64_t)d.heads * (d.dim + d.rot_dim));
       w.qa = std::max<int64_t>(w.qa, (int64_t)d.heads * RP);
       w.olat = std::max<int64_t>(w.olat, (int64_t)d.heads * d.kv_rank);
+      if (d.q_rank == 0 && b200q_latent_expand_ok(d.heads, d.dim, d.rot_dim, d.vdim, d.kv_rank, c.block_size, c.dtype)) {
+        w.lat = std::max<int64_t>(w.lat, d.kv_rank);
+        w.lat_k = std::max<int64_t>(w.lat_k, (int64_t)d.heads * d.dim);
+        w.lat_v = std::max<int64_t>(w.lat_v, (int64_t)d.heads * d.vdim);
+      }
       w.attn = std::max<int64_t>(w.attn, (int64_t)d.heads * d.vdim);
     } else if (d.mixer == B200Q_MIXER_GENERAL_DELTA) {
       w.proj = std::max<int64_t>(w.proj, 5 * (int64_t)d.heads * d.dim + d.decay_rank);
@@ -432,6 +437,11 @@ int64_t layout(b200q_model* m, uint8_t* base) {
   y->blend = take(w.blend ? T * w.blend * es : 1);
   y->tg = take(c.side_dim > 0 ? T * c.side_dim * es : 1);
   y->ta = take(c.side_dim > 0 ? T * c.side_dim * es : 1);
+  y->lat_cap = w.lat_k > 0 ? 2 * T + 1024 : 0;
+  y->lat_rows = take(w.lat_k > 0 ? y->lat_cap * w.lat * es : 1);
+  y->lat_k = take(w.lat_k > 0 ? y->lat_cap * w.lat_k * es : 1);
+  y->lat_v = take(w.lat_k > 0 ? y->lat_cap * w.lat_v * es : 1);
+  y->lat_span = (int32_t*)take(w.lat_k > 0 ? (int64_t)c.max_seqs * 8 : 1);
   y->rot = (float*)take(w.rot ? T * w.rot * 4 : 1);
   y->sel = take(LR * W * es);
   y->logits = (float*)take(LR * (int64_t)c.vocab * 4);
@@ -778,6 +788,7 @@ int layered_bind_weight(b200q_model* m, const char* name, const void* p, int64_t
     }
     if (d.kv_from < 0) FIELD("mix.kv_norm", l.kv_norm, 1, d.kv_rank)
     if (d.sink) FIELD("mix.sink", l.sink, 1, d.heads)
+    if (d.q_rank == 0) FIELD("mix.uk", l.uk, (int64_t)d.heads * d.dim, d.kv_rank)
     FIELD("mix.uk_t", l.uk_t, (int64_t)d.heads * d.kv_rank, d.dim)
     FIELD("mix.uv", l.uv, (int64_t)d.heads * d.vdim, d.kv_rank)
     FIELD("mix.o", l.o, W, (int64_t)d.heads * d.vdim)
@@ -1073,7 +1084,7 @@ int layered_forward(b200q_model* m, const b200q_batch* b, void* stream) {
                                  b->n_rows, T, H, G, d.dim, d.vdim, c.block_size, d.window, d.keep_first, d.softcap,
                                  d.sink ? l.sink : nullptr,
                                  d.bare && !d.channel_gate ? nullptr : (uint8_t*)y->proj + (size_t)(HD + n_kv) * es, NP,
-                                 d.channel_gate, y->attn, dt, stream));
+                                 d.channel_gate, b->max_portion, y->attn, dt, stream));
       return product(y->attn, l.o, outp, HV);  // the output bias, if any, joins in the layer's sum
     }
     return B200Q_OK;
@@ -1119,20 +1130,51 @@ int layered_forward(b200q_model* m, const b200q_batch* b, void* stream) {
       if (!d.rot_half)
         TRY(EW, (double)T * H * P * (es + 4),
             b200q_rope_pairs_q_ex(q, ldq, H, d.dim, P, d.rot_dims, l.freq, l.mag, b->positions, y->qa, R, T, dt, stream));
-      // the unrotated query of every head, carried into the latent space: qa[t,h,:R] = W_uk[h]^T q[t,h,:dim]
-      if (d.dim > 0)
-        TRY(B200Q_PROF_GEMM, 2.0 * T * H * (double)R * d.dim,
-            b200q_linear_batched(q, ldq, QD, l.uk_t, (long long)R * d.dim, y->qa, H * RP, RP, T, R, d.dim, H, dt, 1,
-                                 stream));
-      else
-        B200Q_CUDA(cudaMemset2DAsync(y->qa, (size_t)RP * 4, 0, (size_t)R * 4, (size_t)T * H, cst));
-      TRY(B200Q_PROF_DECODE_ATTN, 0.0,
-          b200q_latent_attn_sink(y->qa, cache, b->block_table, b->bt_stride, b->row_seq, b->positions, T, H, R, P,
-                                 c.block_size, d.window, d.attn_scale, d.sink ? l.sink : nullptr, gate, ldq, y->olat, dt,
-                                 stream));
-      TRY(B200Q_PROF_GEMM, 2.0 * T * H * (double)R * d.vdim,
-          b200q_linear_batched(y->olat, H * R, R, l.uv, (long long)d.vdim * R, y->attn, H * d.vdim, d.vdim, T, d.vdim, R,
-                               H, dt, 0, stream));
+      // Portions of prompts: where every latent they see meets enough of their tokens, the latents are expanded to keys and
+      // values once; single tokens (rows [0, n_dec) of the step) and the other portions stay in the latent space.
+      int rows = 0, longest_span = 0, absorbed = T;
+      if (y->lat_cap > 0 && l.uk && b->h_seq_desc && T > b->n_dec &&
+          b200q_latent_expand_ok(H, d.dim, P, d.vdim, R, c.block_size, dt)) {
+        double meets = 0.0;
+        for (int s = b->n_dec; s < b->n_rows; ++s) {
+          const int n = b->h_seq_desc[4 * s + 1], pos0 = b->h_seq_desc[4 * s + 2];
+          const int span = pos0 + n - (d.window > 0 ? std::max(0, pos0 - d.window + 1) : 0);
+          rows += span;
+          longest_span = std::max(longest_span, span);
+          meets += (double)n * span;
+        }
+        if (rows <= y->lat_cap && meets >= 8.0 * rows) absorbed = b->n_dec;
+      }
+      if (absorbed < T) {
+        TRY(EW, 2.0 * rows * R * es,
+            b200q_latent_gather(cache, b->block_table, b->bt_stride, b->seq_desc, b->n_rows, longest_span, d.window, c.block_size,
+                                R, P, (int)y->lat_cap, y->lat_rows, y->lat_span, stream));
+        TRY(B200Q_PROF_GEMM, 2.0 * rows * H * (double)R * d.dim,
+            b200q_linear(y->lat_rows, R, l.uk, nullptr, y->lat_k, H * d.dim, rows, H * d.dim, R, dt, 0, stream));
+        TRY(B200Q_PROF_GEMM, 2.0 * rows * H * (double)R * d.vdim,
+            b200q_linear(y->lat_rows, R, l.uv, nullptr, y->lat_v, H * d.vdim, rows, H * d.vdim, R, dt, 0, stream));
+        TRY(B200Q_PROF_DECODE_ATTN, 0.0,
+            b200q_latent_portion_attn(q, ldq, y->qa, y->lat_k, y->lat_v, y->lat_span, cache, b->block_table, b->bt_stride,
+                                      b->seq_desc, b->n_rows, b->max_portion > 0 ? b->max_portion : T, H, d.dim, P, d.vdim, R,
+                                      c.block_size, d.window, d.attn_scale, d.sink ? l.sink : nullptr, gate, ldq, y->attn,
+                                      stream));
+      }
+      if (absorbed > 0) {
+        // the unrotated query of every head, carried into the latent space: qa[t,h,:R] = W_uk[h]^T q[t,h,:dim]
+        if (d.dim > 0)
+          TRY(B200Q_PROF_GEMM, 2.0 * absorbed * H * (double)R * d.dim,
+              b200q_linear_batched(q, ldq, QD, l.uk_t, (long long)R * d.dim, y->qa, H * RP, RP, absorbed, R, d.dim, H, dt, 1,
+                                   stream));
+        else
+          B200Q_CUDA(cudaMemset2DAsync(y->qa, (size_t)RP * 4, 0, (size_t)R * 4, (size_t)absorbed * H, cst));
+        TRY(B200Q_PROF_DECODE_ATTN, 0.0,
+            b200q_latent_attn_sink(y->qa, cache, b->block_table, b->bt_stride, b->row_seq, b->positions, absorbed, H, R, P,
+                                   c.block_size, d.window, d.attn_scale, d.sink ? l.sink : nullptr, gate, ldq, y->olat, dt,
+                                   stream));
+        TRY(B200Q_PROF_GEMM, 2.0 * absorbed * H * (double)R * d.vdim,
+            b200q_linear_batched(y->olat, H * R, R, l.uv, (long long)d.vdim * R, y->attn, H * d.vdim, d.vdim, absorbed, d.vdim,
+                                 R, H, dt, 0, stream));
+      }
       return product(y->attn, l.o, y->mix, H * d.vdim);
     } else if (d.mixer == B200Q_MIXER_GENERAL_DELTA) {
       const int HD = d.heads * d.dim, NP = 5 * HD + d.decay_rank;

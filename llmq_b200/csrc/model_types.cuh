@@ -49,6 +49,7 @@ struct b200q_layered_layer {
   const float *in_b = nullptr, *out_b = nullptr, *map_lambda = nullptr;
   // softmax sink per head; the vector a pass begins with; the layer's place among the step's rotation tables (floats per token)
   const float *sink = nullptr, *step = nullptr;
+  const void* uk = nullptr;  // latent attention: the key up-projection as it is (prompt portions expand the latents)
   bool rot_table = false, rot_shared = false;
   int64_t rot_off = 0;
   float mag = 1.f;  // factor of sine and cosine (YaRN)
@@ -89,6 +90,9 @@ struct b200q_layered {
   const void* tok_embed = nullptr;
   int64_t tok_cols = 0;
   void *tg = nullptr, *ta = nullptr;
+  void *lat_rows = nullptr, *lat_k = nullptr, *lat_v = nullptr;  // latents a step's portions see, and their keys and values
+  int32_t* lat_span = nullptr;
+  int64_t lat_cap = 0;   // rows of the three
   float* rot = nullptr;  // cosines and sines of the step's positions, shared by layers of equal rotation
 };
 

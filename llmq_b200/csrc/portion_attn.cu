@@ -1,0 +1,443 @@
+// portion_attn.cu — softmax attention of prompt portions on the tensor cores (bf16 caches): 64 consecutive tokens of a
+// sequence's portion and one head per CTA, keys in tiles of 64.  Two sources of keys and values share the kernel:
+//   grouped-query attention   both from the paged cache ([kv_heads*dim | kv_heads*vdim] rows)
+//   latent attention          the unrotated keys and the values as rows that were expanded from the cached latents for the
+//                             sequence's visible span, the rotated key part from the paged cache.  A prompt reads every
+//                             expanded row many times, so expanding it once costs less than carrying every query into the
+//                             latent space (which single tokens do): per score dim + rot_dim + vdim products instead of
+//                             2 kv_rank + rot_dim.
+// Scores, softmax state and accumulators are fp32; queries and weights are rounded to bf16 as the products see them.
+#include <stdlib.h>
+
+#include <algorithm>
+
+#include "layered_common.cuh"
+
+namespace b200q {
+
+struct SeqView {
+  int row0, n, pos0, slot;
+};
+__device__ __forceinline__ SeqView seq_view(const int32_t* __restrict__ seq_desc, int s) {
+  const int4 v = *reinterpret_cast<const int4*>(seq_desc + 4 * s);
+  return {v.x, v.y, v.z, v.w};
+}
+// keys lo .. pos0 + n - 1 are what a portion's tokens see
+__device__ __forceinline__ int span_begin(const SeqView& s, int window) {
+  return window > 0 ? max(0, s.pos0 - window + 1) : 0;
+}
+
+// 16 bytes into shared memory, zeros when `on` is false
+__device__ __forceinline__ void cp_async16_zfill(void* dst, const void* src, bool on) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(on ? 16 : 0) : "memory");
+}
+
+// ------------------------------------------------------------------------------------------------
+// the latents a step's portions see, gathered from their pages into dense rows (sequence by sequence, in order of the
+// positions), and where each sequence's rows begin: span[s] = {first row, first position}.  CTA = 64 rows of a sequence.
+// ------------------------------------------------------------------------------------------------
+__global__ void __launch_bounds__(256) latent_gather_kernel(const bf16* __restrict__ cache, const int32_t* __restrict__ block_table,
+                                                            int bt_stride, const int32_t* __restrict__ seq_desc, int window,
+                                                            int bs_shift, int R, int RP, int cap, bf16* __restrict__ out,
+                                                            int2* __restrict__ span) {
+  __shared__ int part[8];
+  const SeqView s = seq_view(seq_desc, blockIdx.x);
+  if (s.n <= 1) return;
+  int before = 0;
+  for (int i = threadIdx.x; i < (int)blockIdx.x; i += 256) {
+    const SeqView o = seq_view(seq_desc, i);
+    if (o.n > 1) before += o.pos0 + o.n - span_begin(o, window);
+  }
+  before = __reduce_add_sync(0xffffffffu, before);
+  if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = before;
+  __syncthreads();
+  before = 0;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) before += part[i];
+  const int lo = span_begin(s, window), count = s.pos0 + s.n - lo;
+  if (blockIdx.y == 0 && threadIdx.x == 0) span[blockIdx.x] = make_int2(before, lo);
+  const int32_t* bt = block_table + (long long)blockIdx.x * bt_stride;
+  const int per = R / 8, mask = (1 << bs_shift) - 1;
+  for (int e = threadIdx.x; e < 64 * per; e += 256) {
+    const int r = blockIdx.y * 64 + e / per, c = (e % per) * 8;
+    if (r >= count || before + r >= cap) break;  // (the caller sizes `out` for all rows)
+    const int pos = lo + r;
+    const long long row = ((long long)bt[pos >> bs_shift] << bs_shift) + (pos & mask);
+    st_v4(out + (long long)(before + r) * R + c, ld_v4(cache + row * RP + c));
+  }
+}
+
+struct PortionAttn {
+  const float* q32;   // grouped-query: [T, heads, dim], scale folded in; latent: [T, heads, kv_rank + rot_dim], rotated parts
+  const bf16* q16;    // latent: rows of stride ldq, head h's unrotated query at h * (dim + rot_dim)
+  const bf16* cache;  // paged rows of `row` elements
+  const bf16 *kx, *vx;  // latent: expanded keys [rows][heads*dim] and values [rows][heads*vdim]
+  const int2* span;
+  const int32_t *block_table, *seq_desc;
+  const float* sink;
+  const bf16* gate;
+  bf16* out;  // [T, heads*vdim]
+  float qmul;         // what turns a stored query into one whose scores are in base 2
+  int bt_stride, heads, kv_heads, dim, rot_dim, kv_rank, row, ldq, bs_shift, window, ld_gate, channel_gate, skip_single;
+};
+
+// ------------------------------------------------------------------------------------------------
+// 4 warps of 16 tokens; a tile's rows lie in shared memory with their 16-byte pieces permuted (piece ^ (row & 7)), so
+// ldmatrix meets no bank conflicts without padding.  Eight threads copy 128 bytes of a row side by side; the page
+// numbers of the tile after the next are read one tile ahead.  Late tokens (the longest rows) are launched first.
+// ------------------------------------------------------------------------------------------------
+constexpr int PATT_KEYS = 64;
+constexpr float PATT_NEG = -1e30f;  // finite floor of the running maximum: exp2(masked - floor) = 0, never NaN
+template <int DK, int DV, bool LATENT>
+__global__ void __launch_bounds__(128, 2) portion_attn_kernel(const PortionAttn a) {
+  extern __shared__ __align__(128) uint8_t smraw[];
+  bf16* kbuf = reinterpret_cast<bf16*>(smraw);      // [2][64][DK]
+  bf16* vbuf = kbuf + 2 * PATT_KEYS * DK;           // [2][64][DV]
+  const SeqView sq = seq_view(a.seq_desc, blockIdx.x);
+  const int r0 = (gridDim.z - 1 - blockIdx.z) * 64;
+  if (r0 >= sq.n || (a.skip_single && sq.n == 1)) return;
+  const int nrows = min(64, sq.n - r0), h = blockIdx.y, g = h / (a.heads / a.kv_heads);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gq = lane >> 2, q4 = lane & 3;
+  const int p_first = sq.pos0 + r0, p_last = p_first + nrows - 1;
+  const int lo = a.window > 0 ? max(0, p_first - a.window + 1) : 0;
+  const int ntiles = (p_last - lo) / PATT_KEYS + 1;
+  const int32_t* bt = a.block_table + (long long)blockIdx.x * a.bt_stride;
+  const int page_mask = (1 << a.bs_shift) - 1;
+  int2 sp = make_int2(0, 0);
+  if (LATENT) sp = a.span[blockIdx.x];
+  // this thread copies pieces (tid & 7), + 8, ... of rows tid / 8 + 16 i of a tile
+  const int cr = tid >> 3, cc = tid & 7;
+  int page[4];
+  auto look_up = [&](int c) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) page[i] = bt[min(lo + c * PATT_KEYS + cr + 16 * i, p_last) >> a.bs_shift];
+  };
+  auto load_tile = [&](int c, int buf) {
+    bf16* kb = kbuf + buf * PATT_KEYS * DK;
+    bf16* vb = vbuf + buf * PATT_KEYS * DV;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int r = cr + 16 * i, j = lo + c * PATT_KEYS + r, pos = min(j, p_last);
+      const bool on = j <= p_last;  // rows behind the last token are zeros
+      const bf16* row = a.cache + (((long long)page[i] << a.bs_shift) + (pos & page_mask)) * a.row;
+      const bf16 *k0, *k1 = nullptr, *v0;
+      if (LATENT) {
+        const long long x = sp.x + (pos - sp.y);
+        k0 = a.kx + (x * a.heads + h) * a.dim;
+        k1 = row + a.kv_rank - a.dim;  // rotated part: columns dim .. DK - 1 of the key
+        v0 = a.vx + (x * a.heads + h) * DV;
+      } else {
+        k0 = row + g * DK;
+        v0 = row + a.kv_heads * DK + g * DV;
+      }
+#pragma unroll
+      for (int k = 0; k < DK / 64; ++k) {
+        const int p = cc + 8 * k;
+        cp_async16_zfill(kb + r * DK + ((p ^ (r & 7)) << 3), (LATENT && p * 8 >= a.dim ? k1 : k0) + p * 8, on);
+      }
+#pragma unroll
+      for (int k = 0; k < DV / 64; ++k) {
+        const int p = cc + 8 * k;
+        cp_async16_zfill(vb + r * DV + ((p ^ (r & 7)) << 3), v0 + p * 8, on);
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  // queries into the second key buffer, then into registers; rows past the portion are zeros
+  look_up(0);
+  load_tile(0, 0);
+  {
+    bf16* qb = kbuf + PATT_KEYS * DK;
+    for (int e = tid; e < 64 * (DK / 8); e += 128) {
+      const int r = e / (DK / 8), p = e % (DK / 8);
+      uint4 w = make_uint4(0, 0, 0, 0);
+      if (r < nrows) {
+        const long long th = (long long)(sq.row0 + r0 + r) * a.heads + h;
+        float v[8];
+        if (LATENT && p * 8 < a.dim) {
+          const uint4 x = ld_v4(a.q16 + (long long)(sq.row0 + r0 + r) * a.ldq + (long long)h * (a.dim + a.rot_dim) + p * 8);
+          const uint32_t xw[4] = {x.x, x.y, x.z, x.w};
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            v[2 * i] = bf16_lo(xw[i]);
+            v[2 * i + 1] = bf16_hi(xw[i]);
+          }
+        } else {
+          const float* src = LATENT ? a.q32 + th * (a.kv_rank + a.rot_dim) + a.kv_rank + p * 8 - a.dim : a.q32 + th * DK + p * 8;
+          const float4 x = *reinterpret_cast<const float4*>(src), y = *reinterpret_cast<const float4*>(src + 4);
+          v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
+          v[4] = y.x; v[5] = y.y; v[6] = y.z; v[7] = y.w;
+        }
+        w = make_uint4(pack_bf16x2(v[0] * a.qmul, v[1] * a.qmul), pack_bf16x2(v[2] * a.qmul, v[3] * a.qmul),
+                       pack_bf16x2(v[4] * a.qmul, v[5] * a.qmul), pack_bf16x2(v[6] * a.qmul, v[7] * a.qmul));
+      }
+      st_v4(qb + r * DK + ((p ^ (r & 7)) << 3), w);
+    }
+  }
+  __syncthreads();
+  const int swz = lane & 7;
+  uint32_t qf[DK / 16][4];
+  {
+    const uint32_t q_s = smem_u32(kbuf + PATT_KEYS * DK + (warp * 16 + (lane & 15)) * DK);
+#pragma unroll
+    for (int ks = 0; ks < DK / 16; ++ks)
+      ldsm_x4(q_s + (uint32_t)(((ks * 2 + (lane >> 4)) ^ swz) << 4), qf[ks][0], qf[ks][1], qf[ks][2], qf[ks][3]);
+  }
+  const int krow = (lane & 7) + 8 * (lane >> 4), kck = (lane >> 3) & 1;
+  const int vrow = ((lane >> 3) & 1) * 8 + (lane & 7), vck = lane >> 4;
+  int p_row[2], lo_row[2];
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    const int i = warp * 16 + gq + 8 * r;
+    p_row[r] = i < nrows ? p_first + i : -1;  // a dead row sees no key
+    lo_row[r] = a.window > 0 ? p_row[r] - a.window + 1 : 0;
+  }
+  const int w_first = p_first + warp * 16, w_last = min(w_first + 15, p_last);
+  const int w_lo = a.window > 0 ? w_last - a.window + 1 : 0;  // first key that the warp's last token sees
+  const bool warp_live = warp * 16 < nrows;
+  float m_[2] = {PATT_NEG, PATT_NEG}, l_[2] = {0.f, 0.f};
+  if (a.sink) {  // counted once per row: by the first of the four threads that share it
+    m_[0] = m_[1] = a.sink[h] * 1.4426950408889634f;
+    if (q4 == 0) l_[0] = l_[1] = 1.f;
+  }
+  float o[DV / 8][4];
+#pragma unroll
+  for (int i = 0; i < DV / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  if (ntiles > 1) look_up(1);
+  for (int c = 0; c < ntiles; ++c) {
+    const int buf = c & 1, j0 = lo + c * PATT_KEYS;
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();  // tile c is whole for everyone, tile c - 1 (first time: the queries) is done with
+    if (c + 1 < ntiles) {
+      load_tile(c + 1, buf ^ 1);
+      if (c + 2 < ntiles) look_up(c + 2);
+    }
+    if (!warp_live || j0 > w_last || (a.window > 0 && j0 + PATT_KEYS - 1 < w_first - a.window + 1)) continue;
+    const uint32_t kb_s = smem_u32(kbuf + buf * PATT_KEYS * DK), vb_s = smem_u32(vbuf + buf * PATT_KEYS * DV);
+    float s[8][4];
+#pragma unroll
+    for (int nt = 0; nt < 8; ++nt) s[nt][0] = s[nt][1] = s[nt][2] = s[nt][3] = 0.f;
+#pragma unroll
+    for (int ks = 0; ks < DK / 16; ++ks) {
+      const uint32_t kp = kb_s + (uint32_t)(krow * DK * 2) + (uint32_t)(((ks * 2 + kck) ^ swz) << 4);
+#pragma unroll
+      for (int nt2 = 0; nt2 < 4; ++nt2) {
+        uint32_t b0, b1, b2, b3;
+        ldsm_x4(kp + (uint32_t)(nt2 * 16 * DK * 2), b0, b1, b2, b3);
+        mma_bf16_16816(s[2 * nt2], qf[ks][0], qf[ks][1], qf[ks][2], qf[ks][3], b0, b1);
+        mma_bf16_16816(s[2 * nt2 + 1], qf[ks][0], qf[ks][1], qf[ks][2], qf[ks][3], b2, b3);
+      }
+    }
+    if (j0 + PATT_KEYS - 1 > w_first || nrows < 64 || j0 < w_lo) {
+#pragma unroll
+      for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int j = j0 + nt * 8 + 2 * q4 + (e & 1);
+          if (j > p_row[e >> 1] || j < lo_row[e >> 1]) s[nt][e] = -INFINITY;
+        }
+    }
+    uint32_t pk[16];
+    float corr[2];
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      float mx = PATT_NEG;
+#pragma unroll
+      for (int nt = 0; nt < 8; ++nt) mx = fmaxf(mx, fmaxf(s[nt][2 * r], s[nt][2 * r + 1]));
+      mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+      mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+      const float mn = fmaxf(m_[r], mx);
+      corr[r] = exp2f(m_[r] - mn);
+      m_[r] = mn;
+      float ps = 0.f;
+#pragma unroll
+      for (int nt = 0; nt < 8; ++nt) {
+        const uint32_t v = pack_bf16x2(exp2f(s[nt][2 * r] - mn), exp2f(s[nt][2 * r + 1] - mn));  // masked: exp2(-inf) = 0
+        ps += bf16_lo(v) + bf16_hi(v);
+        pk[(nt >> 1) * 4 + (nt & 1) * 2 + r] = v;
+      }
+      l_[r] = l_[r] * corr[r] + ps;
+    }
+    if (__any_sync(0xffffffffu, corr[0] != 1.f || corr[1] != 1.f)) {
+#pragma unroll
+      for (int i = 0; i < DV / 8; ++i) {
+        o[i][0] *= corr[0];
+        o[i][1] *= corr[0];
+        o[i][2] *= corr[1];
+        o[i][3] *= corr[1];
+      }
+    }
+#pragma unroll
+    for (int kk = 0; kk < 4; ++kk) {
+      const uint32_t vp = vb_s + (uint32_t)((kk * 16 + vrow) * DV * 2);
+#pragma unroll
+      for (int nd = 0; nd < DV / 16; ++nd) {
+        uint32_t b0, b1, b2, b3;
+        ldsm_x4_t(vp + (uint32_t)(((nd * 2 + vck) ^ swz) << 4), b0, b1, b2, b3);
+        mma_bf16_16816(o[2 * nd], pk[4 * kk], pk[4 * kk + 1], pk[4 * kk + 2], pk[4 * kk + 3], b0, b1);
+        mma_bf16_16816(o[2 * nd + 1], pk[4 * kk], pk[4 * kk + 1], pk[4 * kk + 2], pk[4 * kk + 3], b2, b3);
+      }
+    }
+  }
+  if (!warp_live) return;
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    float l = l_[r];
+    l += __shfl_xor_sync(0xffffffffu, l, 1);
+    l += __shfl_xor_sync(0xffffffffu, l, 2);
+    if (p_row[r] < 0) continue;
+    const long long t = sq.row0 + (p_row[r] - sq.pos0);
+    const float gv = a.gate && !a.channel_gate ? sigmoidf_(__bfloat162float(a.gate[t * a.ld_gate + h])) : 1.f;
+    const float inv = gv / l;
+    bf16* orow = a.out + (t * a.heads + h) * DV;
+    const bf16* grow = a.channel_gate ? a.gate + t * a.ld_gate + (long long)h * DV : nullptr;
+#pragma unroll
+    for (int nt = 0; nt < DV / 8; ++nt) {
+      const int d = nt * 8 + 2 * q4;
+      float g0 = 1.f, g1 = 1.f;
+      if (grow) {
+        g0 = sigmoidf_(__bfloat162float(grow[d]));
+        g1 = sigmoidf_(__bfloat162float(grow[d + 1]));
+      }
+      *reinterpret_cast<uint32_t*>(orow + d) = pack_bf16x2(o[nt][2 * r] * inv * g0, o[nt][2 * r + 1] * inv * g1);
+    }
+  }
+}
+
+static int shift_of(int block_size) {  // -1: not a power of two
+  int s = 0;
+  while ((1 << s) < block_size) ++s;
+  return (1 << s) == block_size ? s : -1;
+}
+
+template <int DK, int DV, bool LATENT>
+static int launch_portions(const PortionAttn& a, int n_seqs, int longest, cudaStream_t st) {
+  dim3 grid(n_seqs, a.heads, (longest + 63) / 64);
+  B200Q_CHECK_ARG(grid.y <= 65535 && grid.z <= 65535, "portion_attn: step too large (portions of %d tokens)", longest);
+  constexpr int smem = 2 * PATT_KEYS * (DK + DV) * 2;
+  auto kern = portion_attn_kernel<DK, DV, LATENT>;
+  B200Q_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+  kern<<<grid, 128, smem, st>>>(a);
+  B200Q_LAUNCH_CHECK();
+  return B200Q_OK;
+}
+
+static bool portion_attn_on() {  // B200Q_PORTION_ATTN=0: the kernels it replaces
+  static const bool on = [] {
+    const char* v = getenv("B200Q_PORTION_ATTN");
+    return !v || atoi(v) != 0;
+  }();
+  return on;
+}
+
+bool portion_attn_gqa_ok(const float* qs, const void* cache, const void* out, int kv_heads, int dim, int vdim, int block_size) {
+  return portion_attn_on() && (dim == 64 || dim == 128) && (vdim == 64 || vdim == 128) && shift_of(block_size) >= 0 &&
+         ((reinterpret_cast<uintptr_t>(qs) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(out)) & 15) == 0 &&
+         kv_heads > 0;
+}
+
+int portion_attn_gqa(const float* qs, const void* cache, const int32_t* block_table, int bt_stride, const int32_t* seq_desc,
+                     int n_seqs, int longest, int heads, int kv_heads, int dim, int vdim, int block_size, int window,
+                     const float* sink, const void* gate, int ld_gate, int channel_gate, int skip_single, void* out,
+                     cudaStream_t st) {
+  PortionAttn a{};
+  a.q32 = qs;
+  a.cache = (const bf16*)cache;
+  a.block_table = block_table;
+  a.seq_desc = seq_desc;
+  a.sink = sink;
+  a.gate = (const bf16*)gate;
+  a.out = (bf16*)out;
+  a.qmul = 1.4426950408889634f;
+  a.bt_stride = bt_stride;
+  a.heads = heads;
+  a.kv_heads = kv_heads;
+  a.dim = dim;
+  a.row = kv_heads * (dim + vdim);
+  a.bs_shift = shift_of(block_size);
+  a.window = window;
+  a.ld_gate = ld_gate;
+  a.channel_gate = channel_gate;
+  a.skip_single = skip_single;
+  if (dim == 64) return vdim == 64 ? launch_portions<64, 64, false>(a, n_seqs, longest, st) : launch_portions<64, 128, false>(a, n_seqs, longest, st);
+  return vdim == 64 ? launch_portions<128, 64, false>(a, n_seqs, longest, st) : launch_portions<128, 128, false>(a, n_seqs, longest, st);
+}
+
+}  // namespace b200q
+
+using namespace b200q;
+
+extern "C" {
+
+int b200q_latent_expand_ok(int heads, int dim, int rot_dim, int vdim, int kv_rank, int block_size, int dtype) {
+  const int dk = dim + rot_dim;
+  return dtype == B200Q_DTYPE_BF16 && portion_attn_on() && heads > 0 && (dk == 64 || dk == 128 || dk == 192) && dim > 0 &&
+                 dim % 8 == 0 && (vdim == 64 || vdim == 128) && kv_rank % 64 == 0 && (heads * dim) % 64 == 0 &&
+                 shift_of(block_size) >= 0
+             ? 1
+             : 0;
+}
+
+int b200q_latent_gather(const void* cache, const int32_t* block_table, int bt_stride, const int32_t* seq_desc, int n_seqs,
+                        int longest_span, int window, int block_size, int kv_rank, int rot_dim, int max_rows, void* out,
+                        int32_t* span, void* stream) {
+  B200Q_CHECK_ARG(cache && block_table && seq_desc && out && span && n_seqs > 0 && longest_span > 0 && window >= 0 &&
+                      kv_rank > 0 && kv_rank % 8 == 0 && rot_dim >= 0 && rot_dim % 8 == 0 && shift_of(block_size) >= 0 &&
+                      ((reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(out)) & 15) == 0,
+                  "latent_gather: bad argument (kv_rank=%d rot_dim=%d)", kv_rank, rot_dim);
+  dim3 grid(n_seqs, (longest_span + 63) / 64);
+  B200Q_CHECK_ARG(grid.y <= 65535, "latent_gather: span of %d rows too long", longest_span);
+  latent_gather_kernel<<<grid, 256, 0, as_stream(stream)>>>((const bf16*)cache, block_table, bt_stride, seq_desc, window,
+                                                            shift_of(block_size), kv_rank, kv_rank + rot_dim, max_rows,
+                                                            (bf16*)out, (int2*)span);
+  B200Q_LAUNCH_CHECK();
+  return B200Q_OK;
+}
+
+int b200q_latent_portion_attn(const void* q, int ldq, const float* qa, const void* keys, const void* values, const int32_t* span,
+                              const void* cache, const int32_t* block_table, int bt_stride, const int32_t* seq_desc, int n_seqs,
+                              int longest, int heads, int dim, int rot_dim, int vdim, int kv_rank, int block_size, int window,
+                              float scale, const float* sink, const void* gate, int ld_gate, void* out, void* stream) {
+  B200Q_CHECK_ARG(q && qa && keys && values && span && cache && block_table && seq_desc && out && n_seqs > 0 && longest > 0 &&
+                      window >= 0 && b200q_latent_expand_ok(heads, dim, rot_dim, vdim, kv_rank, block_size, B200Q_DTYPE_BF16) &&
+                      ldq % 8 == 0 && (dim + rot_dim) % 8 == 0 && (!gate || ld_gate >= heads) &&
+                      ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(qa) | reinterpret_cast<uintptr_t>(keys) |
+                        reinterpret_cast<uintptr_t>(values) | reinterpret_cast<uintptr_t>(cache)) & 15) == 0,
+                  "latent_portion_attn: bad argument (heads=%d dim=%d rot_dim=%d vdim=%d kv_rank=%d)", heads, dim, rot_dim, vdim,
+                  kv_rank);
+  PortionAttn a{};
+  a.q32 = qa;
+  a.q16 = (const bf16*)q;
+  a.cache = (const bf16*)cache;
+  a.kx = (const bf16*)keys;
+  a.vx = (const bf16*)values;
+  a.span = (const int2*)span;
+  a.block_table = block_table;
+  a.seq_desc = seq_desc;
+  a.sink = sink;
+  a.gate = (const bf16*)gate;
+  a.out = (bf16*)out;
+  a.qmul = (float)(scale * 1.4426950408889634);
+  a.bt_stride = bt_stride;
+  a.heads = heads;
+  a.kv_heads = heads;
+  a.dim = dim;
+  a.rot_dim = rot_dim;
+  a.kv_rank = kv_rank;
+  a.row = kv_rank + rot_dim;
+  a.ldq = ldq;
+  a.bs_shift = shift_of(block_size);
+  a.window = window;
+  a.ld_gate = ld_gate;
+  a.skip_single = 1;
+  cudaStream_t st = as_stream(stream);
+  const int dk = dim + rot_dim;
+#define PORTIONS(DK) \
+  return vdim == 64 ? launch_portions<DK, 64, true>(a, n_seqs, longest, st) : launch_portions<DK, 128, true>(a, n_seqs, longest, st)
+  if (dk == 64) PORTIONS(64);
+  if (dk == 128) PORTIONS(128);
+  PORTIONS(192);
+#undef PORTIONS
+}
+
+}  // extern "C"

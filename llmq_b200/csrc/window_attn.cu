@@ -744,15 +744,15 @@ int b200q_window_attn_ex(const float* qs, const void* cache, const int32_t* bloc
                          int heads, int kv_heads, int dim, int vdim, int block_size, int window, int keep_first,
                          float softcap, const void* gate, int ld_gate, void* out, int dtype, void* stream) {
   return b200q_window_attn_sink(qs, cache, block_table, bt_stride, row_seq, positions, seq_desc, n_seqs, T_, heads, kv_heads,
-                                dim, vdim, block_size, window, keep_first, softcap, nullptr, gate, ld_gate, 0, out, dtype,
+                                dim, vdim, block_size, window, keep_first, softcap, nullptr, gate, ld_gate, 0, 0, out, dtype,
                                 stream);
 }
 
 int b200q_window_attn_sink(const float* qs, const void* cache, const int32_t* block_table, int bt_stride,
                            const int32_t* row_seq, const int32_t* positions, const int32_t* seq_desc, int n_seqs, int T_,
                            int heads, int kv_heads, int dim, int vdim, int block_size, int window, int keep_first,
-                           float softcap, const float* sink, const void* gate, int ld_gate, int channel_gate, void* out,
-                           int dtype, void* stream) {
+                           float softcap, const float* sink, const void* gate, int ld_gate, int channel_gate, int max_portion,
+                           void* out, int dtype, void* stream) {
   B200Q_CHECK_ARG(!channel_gate || (gate && ld_gate >= heads * vdim), "window_attn: a gate per channel needs rows of %d values",
                   heads * vdim);
   B200Q_CHECK_ARG(keep_first >= 0 && softcap >= 0.f, "window_attn: bad kept keys (%d) or soft cap (%g)", keep_first,
@@ -776,7 +776,18 @@ int b200q_window_attn_sink(const float* qs, const void* cache, const int32_t* bl
     const size_t msm = ((size_t)nw * 16 + 2 * WATT_KEYS) * (dim + 8) * 2 + (size_t)2 * WATT_KEYS * (vdim + 8) * 2;
     // single decoded tokens go to the kernel whose rows are the heads of a group (groups of up to 16 heads); a
     // step of single tokens only (T == n_seqs) needs no tile kernel
-    const bool dec = rep <= 16, tiles = !dec || T_ > n_seqs;
+    const bool dec = rep <= 16;
+    bool tiles = !dec || T_ > n_seqs;
+    // portions without kept keys and soft caps: 64 tokens per CTA
+    if (tiles && keep_first == 0 && softcap == 0.f && portion_attn_gqa_ok(qs, cache, out, kv_heads, dim, vdim, block_size)) {
+      int longest = T_ - n_seqs + 1;
+      if (max_portion > 0 && max_portion < longest) longest = max_portion;
+      if (int rc = portion_attn_gqa(qs, cache, block_table, bt_stride, seq_desc, n_seqs, longest, heads, kv_heads, dim, vdim,
+                                    block_size, window, sink, gate, ld_gate, channel_gate, dec ? 1 : 0, out, st))
+        return rc;
+      if (!dec || (long long)n_seqs * longest == T_) return B200Q_OK;  // (portions of one length: no single tokens)
+      tiles = false;
+    }
     const int dkeys = window_attn_decode_keys(dim, vdim);
     const size_t dsm = std::max((size_t)16 * (dim + 8) * 2 + (size_t)WDEC_WARPS * 2 * dkeys * (dim + vdim + 16) * 2,
                                 (size_t)16 * (dim + 8) * 2 + (size_t)WDEC_WARPS * 16 * (vdim + 2) * 4);

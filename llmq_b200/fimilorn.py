@@ -256,8 +256,8 @@ def engine_weights(spec: FimilornSpec, sd: Dict[str, torch.Tensor]) -> Iterable[
     (bound in the model's dtype); 1-D results are vectors and constants (bound as fp32 rows).  Runs of the same
     checkpoint layer yield the SAME tensor objects, which the model uploads once.  Fusions: the projections that read a
     mixer's input become one matrix with zero rows up to a multiple of 64 (retention and attention: q, k, v, gate;
-    latent attention: q, the latent, the shared rotated key); each head's key up-projection is stored transposed (the
-    query is carried into the latent space); gate and up of the dense unit are stacked (interleaved in blocks of 128 rows
+    latent attention: q, the latent, the shared rotated key); each head's key up-projection is stored transposed too (single
+    tokens carry the query into the latent space); gate and up of the dense unit are stacked (interleaved in blocks of 128 rows
     when ff is a multiple of 128); the experts' matrices are stacked, a shared expert of their size as one more."""
     yield "embed", sd["embed"]
     yield "final_norm", sd["final.norm"]
@@ -283,6 +283,7 @@ def _layer_weights(ly: FimilornLayer, sd) -> Iterable[Tuple[str, torch.Tensor]]:
         yield "mix.kv_norm", sd[m + "dkv.norm"]
         uk = sd[m + "uk"].reshape(ly.heads, ly.dim, ly.kv_rank)
         yield "mix.uk_t", uk.transpose(1, 2).reshape(ly.heads * ly.kv_rank, ly.dim)
+        yield "mix.uk", sd[m + "uk"]     # prompts expand the latents they see instead
         yield "mix.uv", sd[m + "uv"]
         yield "mix.sink", sd[m + "sink"].reshape(-1)
     else:

@@ -283,6 +283,7 @@ def engine_weights(spec: KabavikSpec, sd: Dict[str, torch.Tensor]) -> Iterable[T
             yield o + "mix.kv_norm", sd[m + "dkv.norm"]
             uk = sd[m + "uk"].reshape(ly.heads, ly.dim, ly.kv_rank)
             yield o + "mix.uk_t", uk.transpose(1, 2).reshape(ly.heads * ly.kv_rank, ly.dim)
+            yield o + "mix.uk", sd[m + "uk"]     # prompts expand the latents they see instead
             yield o + "mix.uv", sd[m + "uv"]
             yield o + "mix.o", sd[m + "o"]
         else:

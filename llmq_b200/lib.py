@@ -153,6 +153,7 @@ class Batch(C.Structure):
         ("row_seq", C.c_void_p),
         ("no_sampling", C.c_int32),
         ("max_portion", C.c_int32),
+        ("h_seq_desc", C.c_void_p),
     ]
 
 
@@ -309,7 +310,11 @@ SIGNATURES = {
     "b200q_window_attn_prep_tab": (_i, [_vp, _i, _i, _i, _i, _vp, _i, _i, _i, _i, _i, _vp, _vp, _f, _i, _vp, _vp, _f, _vp,
                                         _vp, _i, _i, _vp]),
     "b200q_window_attn_sink": (_i, [_vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _vp, _vp, _i,
-                                    _i, _vp, _i, _vp]),
+                                    _i, _i, _vp, _i, _vp]),
+    "b200q_latent_expand_ok": (_i, [_i, _i, _i, _i, _i, _i, _i]),
+    "b200q_latent_gather": (_i, [_vp, _vp, _i, _vp, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp]),
+    "b200q_latent_portion_attn": (_i, [_vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f,
+                                       _vp, _vp, _i, _vp, _vp]),
     "b200q_latent_prep_tab": (_i, [_vp, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _i, _f, _i, _vp]),
     "b200q_latent_attn_sink": (_i, [_vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _vp, _vp, _i, _vp, _i, _vp]),
     "b200q_moe_route_gated": (_i, [_vp, _vp, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp]),

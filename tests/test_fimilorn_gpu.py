@@ -223,7 +223,7 @@ def test_attention_sinks_gates_edges_pages_and_far_keys(cuda, case, dtype, how):
         o = torch.zeros(c + n, H * V, dtype=tdt, device=cuda)
         L.check(lib.b200q_window_attn_sink(q.data_ptr(), paged.cache.data_ptr(), table.data_ptr(), paged.nb,
                                            row_seq.data_ptr(), pos.data_ptr(), desc.data_ptr(), 1 + c, c + n, H, G, D, V,
-                                           paged.bs, window, 0, 0.0, sd.data_ptr(), gs.data_ptr(), H * V + 6, 1,
+                                           paged.bs, window, 0, 0.0, sd.data_ptr(), gs.data_ptr(), H * V + 6, 1, n,
                                            o.data_ptr(), dt, None))
         torch.cuda.synchronize()
         if c:   # one key of zeros against the sink: 1 / (1 + exp(sink)), half of it behind the gate
@@ -297,6 +297,104 @@ def test_latent_sinks_edges_pages_and_far_keys(cuda, case, dtype, how):
         seen = [m for m in marks if m <= i and (not window or i - m < window)]
         if seen:
             assert abs(float(want[i, 0, 0]) - sum(seen) / len(seen)) < 0.5
+
+
+EXPANDED_CASES = [
+    # (T, H, unrotated, rotated, values, latent size, window, marked keys)
+    (200, 2, 64, 64, 64, 64, 64, [0, 15, 16, 63, 64, 127, 128, 135]),
+    (300, 3, 128, 64, 128, 128, 80, [3, 79, 80, 83, 159, 160, 200]),
+    (256, 8, 40, 24, 64, 64, 0, [5]),                            # a key of 64 whose parts are no multiples of 16
+    (150, 2, 96, 96, 128, 192, 19, [0, 18, 19, 47, 63, 64, 100]),
+]
+
+
+@pytest.mark.parametrize("case", range(len(EXPANDED_CASES)))
+@pytest.mark.parametrize("how", ["whole", "portions"])
+def test_latent_portions_over_expanded_rows(cuda, case, how):
+    """the rows a portion sees are gathered from their pages in order, every sequence's span where it should be; keys of two
+    parts (expanded, and shared in the cache), a dominating key at window, page and tile edges, sinks and gates per head;
+    single tokens of the step are left alone"""
+    L, lib = _ops()
+    T, H, D, P, V, R, window, marks = EXPANDED_CASES[case]
+    assert lib.b200q_latent_expand_ok(H, D, P, V, R, 16, L.DTYPE_BF16) == 1
+    g = torch.Generator().manual_seed(case)
+    u = torch.randn(D + P, generator=g)
+    u = u / u.norm()
+    q = (0.05 * torch.randn(T, H, D + P, generator=g) + 6.0 * u).bfloat16().float()
+    keys = 0.3 * torch.randn(T, H, D + P, generator=g)
+    keys[..., D:] = keys[:, :1, D:]                              # the rotated part is shared by the heads
+    for j in marks:
+        keys[j] = 4.0 * u
+    keys = keys.bfloat16().float()
+    vals = torch.arange(T, dtype=torch.float32)[:, None, None].expand(T, H, V).bfloat16().float()
+    lat = torch.randn(T, R, generator=g).bfloat16().float()
+    gate = torch.randn(T, H + 3, generator=g).bfloat16().float()
+    sink = torch.linspace(-20.0, 21.6, H)
+    want = O.sink_attention(q.double(), keys.double(), vals.double(), O.visible(T, window), 0.9, sink.double())
+    want = want * torch.sigmoid(gate[:, :H].double())[:, :, None]
+    paged = Paged(cuda, torch.cat([lat, keys[:, 0, D:]], 1), torch.ones(R + P), torch.bfloat16, case)
+    sd = sink.to(cuda)
+    for at, n in portions_of(T, how):
+        if n == 1:
+            continue
+        c, row_seq, pos, desc, table = paged.step(at, n, how != "whole")
+        lo = max(0, at - window + 1) if window else 0
+        count = at + n - lo
+        rows = torch.full((T + 64, R), 9.0, dtype=torch.bfloat16, device=cuda)
+        span = torch.full((2 * (c + 1),), -1, dtype=torch.int32, device=cuda)
+        L.check(lib.b200q_latent_gather(paged.cache.data_ptr(), table.data_ptr(), paged.nb, desc.data_ptr(), 1 + c, count, window,
+                                        16, R, P, T + 64, rows.data_ptr(), span.data_ptr(), None))
+        torch.cuda.synchronize()
+        assert span.cpu().tolist() == [-1, -1] * c + [0, lo]
+        assert torch.equal(rows[:count].float().cpu(), lat[lo:lo + count]) and float(rows[count:].float().min()) == 9.0
+        ldq = H * (D + P) + 8
+        q16 = torch.zeros(c + n, ldq, dtype=torch.bfloat16, device=cuda)
+        q16[c:, :H * (D + P)] = q[at:at + n].reshape(n, -1).bfloat16().to(cuda)
+        qa = torch.full((c + n, H, R + P), 1e4, device=cuda)
+        qa[c:, :, R:] = q[at:at + n, :, D:].to(cuda)
+        kx = keys[lo:lo + count, :, :D].bfloat16().to(cuda).contiguous()
+        vx = vals[lo:lo + count].bfloat16().to(cuda).contiguous()
+        gs = torch.zeros(c + n, H + 3, dtype=torch.bfloat16, device=cuda)
+        gs[c:] = gate[at:at + n].bfloat16().to(cuda)
+        o = torch.full((c + n, H * V), 77.0, dtype=torch.bfloat16, device=cuda)
+        L.check(lib.b200q_latent_portion_attn(q16.data_ptr(), ldq, qa.data_ptr(), kx.data_ptr(), vx.data_ptr(), span.data_ptr(),
+                                              paged.cache.data_ptr(), table.data_ptr(), paged.nb, desc.data_ptr(), 1 + c, n, H, D,
+                                              P, V, R, 16, window, 0.9, sd.data_ptr(), gs.data_ptr(), H + 3, o.data_ptr(), None))
+        torch.cuda.synchronize()
+        assert float((o[c:].float().cpu().double().view(n, H, V) - want[at:at + n]).abs().max()) < 2e-2 * T
+        if c:
+            assert float(o[0].float().min()) == 77.0
+    for i in range(T):                                          # the marks do what they are meant to (head 0: no sink)
+        seen = [m for m in marks if m <= i and (not window or i - m < window)]
+        if seen:
+            assert abs(float(want[i, 0, 0] / torch.sigmoid(gate[i, 0].double())) - sum(seen) / len(seen)) < 0.6
+
+
+def test_latent_spans_of_several_portions(cuda):
+    """rows of three portions behind two single tokens: each sequence's rows follow the one before, windows cut them"""
+    L, lib = _ops()
+    R, P, bs = 64, 8, 16
+    cache = torch.randn(40 * bs, R + P).bfloat16()
+    bt = torch.randperm(40)[:35].view(5, 7).to(torch.int32)
+    seqs = [(1, 30), (1, 0), (5, 0), (40, 33), (2, 90)]          # (tokens, position of the first)
+    at, desc = 0, []
+    for i, (n, p0) in enumerate(seqs):
+        desc.append([at, n, p0, i])
+        at += n
+    cd, btd, dd = cache.to(cuda), bt.to(cuda), torch.tensor(desc, dtype=torch.int32, device=cuda)
+    for window in (0, 20):
+        want, spans = [], [[-1, -1], [-1, -1]]
+        for i, (n, p0) in enumerate(seqs[2:], 2):
+            lo = max(0, p0 - window + 1) if window else 0
+            spans.append([len(want), lo])
+            want += [cache[int(bt[i, p // bs]) * bs + p % bs, :R] for p in range(lo, p0 + n)]
+        out = torch.zeros(len(want) + 3, R, dtype=torch.bfloat16, device=cuda)
+        span = torch.full((10,), -1, dtype=torch.int32, device=cuda)
+        L.check(lib.b200q_latent_gather(cd.data_ptr(), btd.data_ptr(), 7, dd.data_ptr(), 5, 100, window, bs, R, P, len(want) + 3,
+                                        out.data_ptr(), span.data_ptr(), None))
+        torch.cuda.synchronize()
+        assert span.cpu().view(5, 2).tolist() == spans
+        assert torch.equal(out.cpu()[:len(want)], torch.stack(want)) and float(out[len(want):].float().abs().max()) == 0.0
 
 
 RETENTION_CASES = [
