@@ -732,7 +732,7 @@ def run_compare(args):
             elif kind in ("attention", "attention_2", "parallel"):
                 per_key = 2.0 * ly.heads * (ly.dim + ly.vdim)
             elif kind == "latent_attention":
-                per_key = 2.0 * ly.heads * (2 * ly.kv_rank + ly.rot_dim)
+                per_key = 2.0 * ly.heads * (ly.dim + ly.rot_dim + ly.vdim)   # over expanded keys and values
             else:
                 continue
             w = getattr(ly, "window", 0) or S_p

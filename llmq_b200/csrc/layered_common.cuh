@@ -38,12 +38,11 @@ static inline int grid_for(long long total, int block = 256) {
   long long g = (total + block - 1) / block;
   return (int)(g < 1 ? 1 : (g > 148 * 16 ? 148 * 16 : g));
 }
-// portion_attn.cu: grouped-query attention of prompt portions on the tensor cores (behind b200q_window_attn_sink)
+// portion_attn.cu: grouped-query attention of a step's portions and single tokens on the tensor cores (behind b200q_window_attn_sink)
 bool portion_attn_gqa_ok(const float* qs, const void* cache, const void* out, int kv_heads, int dim, int vdim, int block_size);
 int portion_attn_gqa(const float* qs, const void* cache, const int32_t* block_table, int bt_stride, const int32_t* seq_desc,
-                     int n_seqs, int longest, int heads, int kv_heads, int dim, int vdim, int block_size, int window,
-                     const float* sink, const void* gate, int ld_gate, int channel_gate, int skip_single, void* out,
-                     cudaStream_t st);
+                     int n_seqs, int longest, int T, int heads, int kv_heads, int dim, int vdim, int block_size, int window,
+                     const float* sink, const void* gate, int ld_gate, int channel_gate, void* out, cudaStream_t st);
 
 static inline bool is_dtype(int d) { return d == B200Q_DTYPE_BF16 || d == B200Q_DTYPE_F32; }
 

@@ -1,4 +1,4 @@
-// portion_attn.cu — softmax attention of prompt portions on the tensor cores (bf16 caches): 64 consecutive tokens of a
+// portion_attn.cu — softmax attention on the tensor cores (bf16 caches).  Prompt portions: 64 consecutive tokens of a
 // sequence's portion and one head per CTA, keys in tiles of 64.  Two sources of keys and values share the kernel:
 //   grouped-query attention   both from the paged cache ([kv_heads*dim | kv_heads*vdim] rows)
 //   latent attention          the unrotated keys and the values as rows that were expanded from the cached latents for the
@@ -6,6 +6,7 @@
 //                             expanded row many times, so expanding it once costs less than carrying every query into the
 //                             latent space (which single tokens do): per score dim + rot_dim + vdim products instead of
 //                             2 kv_rank + rot_dim.
+// Single tokens of grouped-query attention: one CTA per (sequence, key head), below.
 // Scores, softmax state and accumulators are fp32; queries and weights are rounded to bf16 as the products see them.
 #include <stdlib.h>
 
@@ -304,6 +305,196 @@ __global__ void __launch_bounds__(128, 2) portion_attn_kernel(const PortionAttn 
   }
 }
 
+// ------------------------------------------------------------------------------------------------
+// single decoded tokens, grouped-query attention: one CTA per (sequence, key head); the 16 rows of a tile are the heads of
+// the group.  Each warp takes the tiles of 16 keys warp, warp + nw, ... through its own ring of STG stages (no CTA barrier in
+// the loop), the rows of a stage looked up one tile before they are asked for; the warps' states are merged in a fixed
+// order.  nw (2, 4 or 8) is the block's size: many sequences take small blocks, which fit one wave with four per SM.
+// ------------------------------------------------------------------------------------------------
+constexpr int TATT_KEYS = 16, TATT_STG = 3;
+template <int DK, int DV>
+__global__ void __launch_bounds__(256) token_attn_kernel(const PortionAttn a) {
+  extern __shared__ __align__(128) uint8_t smraw[];
+  constexpr int STAGE = TATT_KEYS * (DK + DV);       // elements of a stage: keys, then values
+  constexpr int MS = DV + 2;
+  const SeqView sq = seq_view(a.seq_desc, blockIdx.x);
+  if (sq.n != 1) return;  // portions of prompts take the tile kernel
+  const int nw = blockDim.x >> 5, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gq = lane >> 2, q4 = lane & 3;
+  const int g = blockIdx.y, rep = a.heads / a.kv_heads;
+  bf16* ring = reinterpret_cast<bf16*>(smraw) + (long long)warp * TATT_STG * STAGE;
+  bf16* qb = reinterpret_cast<bf16*>(smraw) + (long long)nw * TATT_STG * STAGE;  // [16][DK]
+  float* mrg = reinterpret_cast<float*>(smraw);                                  // after the loop: [nw][16][DV + 2]
+  const int p = sq.pos0, lo = a.window > 0 ? max(0, p - a.window + 1) : 0;
+  const int ntiles = (p - lo) / TATT_KEYS + 1, n_it = warp < ntiles ? (ntiles - warp + nw - 1) / nw : 0;
+  const long long t = sq.row0;
+  const int32_t* bt = a.block_table + (long long)blockIdx.x * a.bt_stride;
+  const int page_mask = (1 << a.bs_shift) - 1;
+  int row_next = 0;  // lane l (mod 16): cache row of key l of the next tile to be asked for
+  auto look_up = [&](int it) {
+    const int pos = min(lo + (warp + it * nw) * TATT_KEYS + (lane & 15), p);
+    row_next = (bt[pos >> a.bs_shift] << a.bs_shift) + (pos & page_mask);
+  };
+  auto load_tile = [&](int it) {
+    bf16* kb = ring + (it % TATT_STG) * STAGE;
+    const int j0 = lo + (warp + it * nw) * TATT_KEYS;
+    constexpr int PER = (DK + DV) / 8;  // 16-byte pieces of a key and its value
+#pragma unroll
+    for (int i = 0; i < TATT_KEYS * PER / 32; ++i) {
+      const int e = i * 32 + lane, j = e / PER, c = e % PER;
+      const bf16* row = a.cache + (long long)__shfl_sync(0xffffffffu, row_next, j) * a.row;
+      const bool key = c < DK / 8;
+      const int v = c - DK / 8;
+      const bf16* src = key ? row + g * DK + c * 8 : row + a.kv_heads * DK + g * DV + v * 8;
+      bf16* dst = key ? kb + j * DK + ((c ^ (j & 7)) << 3) : kb + TATT_KEYS * DK + j * DV + ((v ^ (j & 7)) << 3);
+      cp_async16_zfill(dst, src, j0 + j <= p);
+    }
+  };
+  auto commit = [&]() { asm volatile("cp.async.commit_group;" ::: "memory"); };
+  if (n_it > 0) look_up(0);
+  for (int i = 0; i < TATT_STG - 1; ++i) {  // every turn commits a group, so that the count of groups is the same for all
+    if (i < n_it) {
+      load_tile(i);
+      if (i + 1 < n_it) look_up(i + 1);
+    }
+    commit();
+  }
+  for (int e = tid; e < 16 * (DK / 8); e += blockDim.x) {
+    const int r = e / (DK / 8), c = e % (DK / 8);
+    uint4 w = make_uint4(0, 0, 0, 0);
+    if (r < rep) {
+      const float* src = a.q32 + (t * a.heads + g * rep + r) * DK + c * 8;
+      const float4 x = *reinterpret_cast<const float4*>(src), y = *reinterpret_cast<const float4*>(src + 4);
+      w = make_uint4(pack_bf16x2(x.x * a.qmul, x.y * a.qmul), pack_bf16x2(x.z * a.qmul, x.w * a.qmul),
+                     pack_bf16x2(y.x * a.qmul, y.y * a.qmul), pack_bf16x2(y.z * a.qmul, y.w * a.qmul));
+    }
+    st_v4(qb + r * DK + ((c ^ (r & 7)) << 3), w);
+  }
+  __syncthreads();
+  const int swz = lane & 7;
+  uint32_t qf[DK / 16][4];
+  {
+    const uint32_t q_s = smem_u32(qb + (lane & 15) * DK);
+#pragma unroll
+    for (int ks = 0; ks < DK / 16; ++ks)
+      ldsm_x4(q_s + (uint32_t)(((ks * 2 + (lane >> 4)) ^ swz) << 4), qf[ks][0], qf[ks][1], qf[ks][2], qf[ks][3]);
+  }
+  const int krow = (lane & 7) + 8 * (lane >> 4), kck = (lane >> 3) & 1;
+  const int vrow = ((lane >> 3) & 1) * 8 + (lane & 7), vck = lane >> 4;
+  float m_[2] = {PATT_NEG, PATT_NEG}, l_[2] = {0.f, 0.f};
+  if (a.sink && warp == 0) {  // counted once: by the first warp's state, there by the first of a row's four threads
+#pragma unroll
+    for (int r = 0; r < 2; ++r)
+      if (gq + 8 * r < rep) {
+        m_[r] = a.sink[g * rep + gq + 8 * r] * 1.4426950408889634f;
+        l_[r] = q4 == 0 ? 1.f : 0.f;
+      }
+  }
+  float o[DV / 8][4];
+#pragma unroll
+  for (int i = 0; i < DV / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  for (int it = 0; it < n_it; ++it) {
+    asm volatile("cp.async.wait_group %0;" ::"n"(TATT_STG - 2) : "memory");
+    __syncwarp();  // tile `it` is whole for the warp; the stage of tile it - 1 is done with
+    if (it + TATT_STG - 1 < n_it) {
+      load_tile(it + TATT_STG - 1);
+      if (it + TATT_STG < n_it) look_up(it + TATT_STG);
+    }
+    commit();
+    const bf16* kb = ring + (it % TATT_STG) * STAGE;
+    const uint32_t kb_s = smem_u32(kb), vb_s = smem_u32(kb + TATT_KEYS * DK);
+    const int j0 = lo + (warp + it * nw) * TATT_KEYS;
+    float s[2][4];
+#pragma unroll
+    for (int nt = 0; nt < 2; ++nt) s[nt][0] = s[nt][1] = s[nt][2] = s[nt][3] = 0.f;
+#pragma unroll
+    for (int ks = 0; ks < DK / 16; ++ks) {
+      uint32_t b0, b1, b2, b3;
+      ldsm_x4(kb_s + (uint32_t)(krow * DK * 2) + (uint32_t)(((ks * 2 + kck) ^ swz) << 4), b0, b1, b2, b3);
+      mma_bf16_16816(s[0], qf[ks][0], qf[ks][1], qf[ks][2], qf[ks][3], b0, b1);
+      mma_bf16_16816(s[1], qf[ks][0], qf[ks][1], qf[ks][2], qf[ks][3], b2, b3);
+    }
+    uint32_t pk[4];
+    float corr[2];
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      float mx = PATT_NEG;
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+          if (gq + 8 * r >= rep || j0 + nt * 8 + 2 * q4 + k > p) s[nt][2 * r + k] = -INFINITY;
+          mx = fmaxf(mx, s[nt][2 * r + k]);
+        }
+      mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+      mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+      const float mn = fmaxf(m_[r], mx);
+      corr[r] = exp2f(m_[r] - mn);
+      m_[r] = mn;
+      float ps = 0.f;
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt) {
+        const uint32_t v = pack_bf16x2(exp2f(s[nt][2 * r] - mn), exp2f(s[nt][2 * r + 1] - mn));
+        ps += bf16_lo(v) + bf16_hi(v);
+        pk[nt * 2 + r] = v;
+      }
+      l_[r] = l_[r] * corr[r] + ps;
+    }
+    if (__any_sync(0xffffffffu, corr[0] != 1.f || corr[1] != 1.f)) {
+#pragma unroll
+      for (int i = 0; i < DV / 8; ++i) {
+        o[i][0] *= corr[0];
+        o[i][1] *= corr[0];
+        o[i][2] *= corr[1];
+        o[i][3] *= corr[1];
+      }
+    }
+    const uint32_t vp = vb_s + (uint32_t)(vrow * DV * 2);
+#pragma unroll
+    for (int nd = 0; nd < DV / 16; ++nd) {
+      uint32_t b0, b1, b2, b3;
+      ldsm_x4_t(vp + (uint32_t)(((nd * 2 + vck) ^ swz) << 4), b0, b1, b2, b3);
+      mma_bf16_16816(o[2 * nd], pk[0], pk[1], pk[2], pk[3], b0, b1);
+      mma_bf16_16816(o[2 * nd + 1], pk[0], pk[1], pk[2], pk[3], b2, b3);
+    }
+    __syncwarp();  // every lane is done with the stage before its next rows are asked for
+  }
+  // ---- merge: [warp][row][DV + 2] = (o..., m, l); a warp without tiles holds (0, floor, 0) ----
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  __syncthreads();  // every warp is done with its ring: it becomes the merge area
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    l_[r] += __shfl_xor_sync(0xffffffffu, l_[r], 1);
+    l_[r] += __shfl_xor_sync(0xffffffffu, l_[r], 2);
+    float* dst = mrg + (long long)(warp * 16 + gq + 8 * r) * MS;
+#pragma unroll
+    for (int nt = 0; nt < DV / 8; ++nt) {
+      dst[nt * 8 + 2 * q4] = o[nt][2 * r];
+      dst[nt * 8 + 2 * q4 + 1] = o[nt][2 * r + 1];
+    }
+    if (q4 == 0) {
+      dst[DV] = m_[r];
+      dst[DV + 1] = l_[r];
+    }
+  }
+  __syncthreads();
+  for (int hh = warp; hh < rep; hh += nw) {  // one warp per head
+    float mx = PATT_NEG, den = 0.f;
+    for (int w = 0; w < nw; ++w) mx = fmaxf(mx, mrg[(long long)(w * 16 + hh) * MS + DV]);
+    for (int w = 0; w < nw; ++w) den = fmaf(mrg[(long long)(w * 16 + hh) * MS + DV + 1], exp2f(mrg[(long long)(w * 16 + hh) * MS + DV] - mx), den);
+    const int h = g * rep + hh;
+    const float gv = a.gate && !a.channel_gate ? sigmoidf_(__bfloat162float(a.gate[t * a.ld_gate + h])) : 1.f;
+    const float inv = gv / den;
+#pragma unroll
+    for (int i = 0; i < DV / 32; ++i) {
+      const int d = lane + 32 * i;
+      float num = 0.f;
+      for (int w = 0; w < nw; ++w) num = fmaf(mrg[(long long)(w * 16 + hh) * MS + d], exp2f(mrg[(long long)(w * 16 + hh) * MS + DV] - mx), num);
+      if (a.channel_gate) num *= sigmoidf_(__bfloat162float(a.gate[t * a.ld_gate + (long long)h * DV + d]));
+      a.out[(t * a.heads + h) * DV + d] = __float2bfloat16_rn(num * inv);
+    }
+  }
+}
+
 static int shift_of(int block_size) {  // -1: not a power of two
   int s = 0;
   while ((1 << s) < block_size) ++s;
@@ -318,6 +509,23 @@ static int launch_portions(const PortionAttn& a, int n_seqs, int longest, cudaSt
   auto kern = portion_attn_kernel<DK, DV, LATENT>;
   B200Q_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
   kern<<<grid, 128, smem, st>>>(a);
+  B200Q_LAUNCH_CHECK();
+  return B200Q_OK;
+}
+
+template <int DK, int DV>
+static int launch_gqa_portions(const PortionAttn& a, int n_seqs, int longest, cudaStream_t st) {
+  return launch_portions<DK, DV, false>(a, n_seqs, longest, st);
+}
+
+template <int DK, int DV>
+static int launch_tokens(const PortionAttn& a, int n_seqs, cudaStream_t st) {
+  const long long blocks = (long long)n_seqs * a.kv_heads;
+  const int nw = blocks > 2 * 148 ? 2 : blocks > 148 ? 4 : 8;
+  const int smem = std::max(nw * TATT_STG * TATT_KEYS * (DK + DV) * 2 + 16 * DK * 2, nw * 16 * (DV + 2) * 4);
+  auto kern = token_attn_kernel<DK, DV>;
+  B200Q_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+  kern<<<dim3(n_seqs, a.kv_heads), nw * 32, smem, st>>>(a);
   B200Q_LAUNCH_CHECK();
   return B200Q_OK;
 }
@@ -337,9 +545,8 @@ bool portion_attn_gqa_ok(const float* qs, const void* cache, const void* out, in
 }
 
 int portion_attn_gqa(const float* qs, const void* cache, const int32_t* block_table, int bt_stride, const int32_t* seq_desc,
-                     int n_seqs, int longest, int heads, int kv_heads, int dim, int vdim, int block_size, int window,
-                     const float* sink, const void* gate, int ld_gate, int channel_gate, int skip_single, void* out,
-                     cudaStream_t st) {
+                     int n_seqs, int longest, int T, int heads, int kv_heads, int dim, int vdim, int block_size, int window,
+                     const float* sink, const void* gate, int ld_gate, int channel_gate, void* out, cudaStream_t st) {
   PortionAttn a{};
   a.q32 = qs;
   a.cache = (const bf16*)cache;
@@ -358,9 +565,18 @@ int portion_attn_gqa(const float* qs, const void* cache, const int32_t* block_ta
   a.window = window;
   a.ld_gate = ld_gate;
   a.channel_gate = channel_gate;
-  a.skip_single = skip_single;
-  if (dim == 64) return vdim == 64 ? launch_portions<64, 64, false>(a, n_seqs, longest, st) : launch_portions<64, 128, false>(a, n_seqs, longest, st);
-  return vdim == 64 ? launch_portions<128, 64, false>(a, n_seqs, longest, st) : launch_portions<128, 128, false>(a, n_seqs, longest, st);
+  const bool tokens = heads / kv_heads <= 16;  // groups of more heads than a tile has rows: the portions' kernel serves all
+  a.skip_single = tokens ? 1 : 0;
+#define BY_SIZE(F, ...)                                                              \
+  (dim == 64 ? (vdim == 64 ? F<64, 64>(__VA_ARGS__) : F<64, 128>(__VA_ARGS__))       \
+             : (vdim == 64 ? F<128, 64>(__VA_ARGS__) : F<128, 128>(__VA_ARGS__)))
+  if (T > n_seqs || !tokens) {
+    if (int rc = BY_SIZE(launch_gqa_portions, a, n_seqs, longest, st)) return rc;
+    if ((long long)n_seqs * longest == T) return B200Q_OK;  // portions of one length: no single tokens
+  }
+  if (!tokens) return B200Q_OK;
+  return BY_SIZE(launch_tokens, a, n_seqs, st);
+#undef BY_SIZE
 }
 
 }  // namespace b200q

@@ -147,6 +147,115 @@ __global__ void __launch_bounds__(128) window_attn_prep_opt_kernel(
     stf(row + GD + e, ldf(pr + v_off + e) + (bias ? bias[v_off + e] : 0.f));
 }
 
+// step 1 from the step's table, 8 values (and their 8 partners where they turn) per thread and unit, one pass over registers:
+// no biases, no temperatures, a norm over the whole projection or none; half a multiple of 8.  Units of a token: the pieces
+// of q's heads, of k's heads, of v.
+constexpr int PREP_UNITS = 2;
+__global__ void __launch_bounds__(256) window_attn_prep_v8_kernel(
+    const bf16* __restrict__ proj, int ldp, int q_off, int k_off, int v_off, int heads, int kv_heads, int dim, int vdim,
+    int qk_norm, const float* __restrict__ w_qn, const float* __restrict__ w_kn, float eps, int half,
+    const float2* __restrict__ table, const int32_t* __restrict__ slot_mapping, float scale, float* __restrict__ qs,
+    bf16* __restrict__ cache) {
+  __shared__ float red[2][8];
+  const long long t = blockIdx.x;
+  const int HD = heads * dim, GD = kv_heads * dim, GV = kv_heads * vdim, per = dim / 8 - half / 8;
+  const int nq = heads * per, nk = k_off >= 0 ? kv_heads * per : 0, nv = k_off >= 0 ? GV / 8 : 0;
+  const bf16* pr = proj + t * ldp;
+  const int slot = k_off >= 0 ? slot_mapping[t] : -1;
+  float a[PREP_UNITS][8], b[PREP_UNITS][8], ss[2] = {0.f, 0.f};
+  int at[PREP_UNITS];  // first value of the unit in its projection; -1: none
+  auto load = [&](const bf16* src, float (&v)[8]) {
+    const uint4 x = ld_v4(src);
+    const uint32_t w[4] = {x.x, x.y, x.z, x.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      v[2 * i] = bf16_lo(w[i]);
+      v[2 * i + 1] = bf16_hi(w[i]);
+    }
+  };
+#pragma unroll
+  for (int q = 0; q < PREP_UNITS; ++q) {
+    const int u = threadIdx.x + 256 * q;
+    at[q] = -1;
+    if (u < nq + nk) {
+      const int w = u < nq ? u : u - nq, piece = w % per;
+      const bool pair = piece < half / 8;
+      at[q] = (w / per) * dim + (pair ? piece * 8 : half + piece * 8);
+      const bf16* src = pr + (u < nq ? q_off : k_off) + at[q];
+      load(src, a[q]);
+      float sum = 0.f;
+#pragma unroll
+      for (int i = 0; i < 8; ++i) sum = fmaf(a[q][i], a[q][i], sum);
+      if (pair) {
+        load(src + half, b[q]);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) sum = fmaf(b[q][i], b[q][i], sum);
+      }
+      ss[u < nq ? 0 : 1] += sum;
+    } else if (u < nq + nk + nv && slot >= 0) {
+      const int c = (u - nq - nk) * 8;
+      st_v4(cache + (long long)slot * (GD + GV) + GD + c, ld_v4(pr + v_off + c));
+    }
+  }
+  float inv[2] = {1.f, 1.f};
+  if (qk_norm) {
+#pragma unroll
+    for (int w = 0; w < 2; ++w) {
+      const float v = warp_sum(ss[w]);
+      if ((threadIdx.x & 31) == 0) red[w][threadIdx.x >> 5] = v;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int w = 0; w < 2; ++w) {
+      float v = 0.f;
+#pragma unroll
+      for (int i = 0; i < 8; ++i) v += red[w][i];
+      inv[w] = 1.f / sqrtf(v / (float)(w ? GD : HD) + eps);
+    }
+  }
+#pragma unroll
+  for (int q = 0; q < PREP_UNITS; ++q) {
+    const int u = threadIdx.x + 256 * q;
+    if (at[q] < 0) continue;
+    const bool is_q = u < nq;
+    if (!is_q && slot < 0) continue;
+    const int d = at[q] % dim;
+    const bool pair = d < half;
+    const float* w = is_q ? w_qn : w_kn;
+    auto finish = [&](float (&v)[8], int off) {
+      if (!qk_norm) return;
+      const float4 x = *reinterpret_cast<const float4*>(w + at[q] + off), y = *reinterpret_cast<const float4*>(w + at[q] + off + 4);
+      const float m = is_q ? inv[0] : inv[1];
+      v[0] *= m * x.x; v[1] *= m * x.y; v[2] *= m * x.z; v[3] *= m * x.w;
+      v[4] *= m * y.x; v[5] *= m * y.y; v[6] *= m * y.z; v[7] *= m * y.w;
+    };
+    auto store = [&](const float (&v)[8], int off) {
+      if (is_q) {
+        float4* o = reinterpret_cast<float4*>(qs + t * HD + at[q] + off);
+        o[0] = make_float4(v[0] * scale, v[1] * scale, v[2] * scale, v[3] * scale);
+        o[1] = make_float4(v[4] * scale, v[5] * scale, v[6] * scale, v[7] * scale);
+      } else {
+        st_v4(cache + (long long)slot * (GD + GV) + at[q] + off,
+              make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7])));
+      }
+    };
+    finish(a[q], 0);
+    if (pair) {
+      finish(b[q], half);
+      const float2* cs = table + t * half + d;
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        const float2 c = cs[i];
+        const float x = a[q][i], y = b[q][i];
+        a[q][i] = x * c.x - y * c.y;
+        b[q][i] = y * c.x + x * c.y;
+      }
+      store(b[q], half);
+    }
+    store(a[q], 0);
+  }
+}
+
 // ------------------------------------------------------------------------------------------------
 // step 2, scalar form: one CTA per (token, key/value head, group of 8 query heads that share it).  Tiles of 32
 // cached keys and values are staged in shared memory once and used by up to 8 query heads (warp = head; lane =
@@ -707,6 +816,22 @@ int b200q_window_attn_prep_tab(const void* proj, int ldp, int q_off, int k_off, 
                                int rot_dims, const float* table, const int32_t* slot_mapping, float scale, float* qs,
                                void* cache, int T_, int dtype, void* stream) {
   B200Q_CHECK_ARG(rot_dims == 0 || table, "window_attn_prep: the table is missing");
+  const bool own = k_off >= 0;
+  const int half = rot_dims / 2, units = (heads + (own ? kv_heads : 0)) * (dim / 8 - half / 8) + (own ? kv_heads * vdim / 8 : 0);
+  if (dtype == B200Q_DTYPE_BF16 && T_ > 0 && !bias && (qk_norm == 0 || qk_norm == 1) && proj && qs && heads > 0 && kv_heads > 0 &&
+      dim > 0 && vdim > 0 && dim % 8 == 0 && vdim % 8 == 0 && rot_dims >= 0 && half % 8 == 0 && 2 * half == rot_dims &&
+      rot_dims <= dim && ldp % 8 == 0 && q_off >= 0 && q_off % 8 == 0 && ldp >= q_off + heads * dim &&
+      (!own || (k_off % 8 == 0 && v_off >= 0 && v_off % 8 == 0 && slot_mapping && cache && ldp >= k_off + kv_heads * dim &&
+                ldp >= v_off + kv_heads * vdim)) &&
+      (qk_norm == 0 || (w_qn && (!own || w_kn))) && units <= 256 * PREP_UNITS &&
+      ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(qs) | reinterpret_cast<uintptr_t>(cache) |
+        reinterpret_cast<uintptr_t>(w_qn) | reinterpret_cast<uintptr_t>(w_kn)) & 15) == 0) {
+    window_attn_prep_v8_kernel<<<T_, 256, 0, as_stream(stream)>>>((const bf16*)proj, ldp, q_off, k_off, v_off, heads, kv_heads, dim,
+                                                                  vdim, qk_norm, w_qn, w_kn, eps, half, (const float2*)table,
+                                                                  slot_mapping, scale, qs, (bf16*)cache);
+    B200Q_LAUNCH_CHECK();
+    return B200Q_OK;
+  }
   return window_attn_prep_any(proj, ldp, q_off, k_off, v_off, bias, heads, kv_heads, dim, vdim, qk_norm, w_qn, w_kn, eps,
                               rot_dims, nullptr, 1.f, (const float2*)table, nullptr, slot_mapping, nullptr, scale, 0.f, 0, qs,
                               cache, T_, dtype, stream);
@@ -776,18 +901,14 @@ int b200q_window_attn_sink(const float* qs, const void* cache, const int32_t* bl
     const size_t msm = ((size_t)nw * 16 + 2 * WATT_KEYS) * (dim + 8) * 2 + (size_t)2 * WATT_KEYS * (vdim + 8) * 2;
     // single decoded tokens go to the kernel whose rows are the heads of a group (groups of up to 16 heads); a
     // step of single tokens only (T == n_seqs) needs no tile kernel
-    const bool dec = rep <= 16;
-    bool tiles = !dec || T_ > n_seqs;
-    // portions without kept keys and soft caps: 64 tokens per CTA
-    if (tiles && keep_first == 0 && softcap == 0.f && portion_attn_gqa_ok(qs, cache, out, kv_heads, dim, vdim, block_size)) {
+    // without kept keys and soft caps: 64 tokens of a portion per CTA, deeper rings for single tokens
+    if (keep_first == 0 && softcap == 0.f && portion_attn_gqa_ok(qs, cache, out, kv_heads, dim, vdim, block_size)) {
       int longest = T_ - n_seqs + 1;
       if (max_portion > 0 && max_portion < longest) longest = max_portion;
-      if (int rc = portion_attn_gqa(qs, cache, block_table, bt_stride, seq_desc, n_seqs, longest, heads, kv_heads, dim, vdim,
-                                    block_size, window, sink, gate, ld_gate, channel_gate, dec ? 1 : 0, out, st))
-        return rc;
-      if (!dec || (long long)n_seqs * longest == T_) return B200Q_OK;  // (portions of one length: no single tokens)
-      tiles = false;
+      return portion_attn_gqa(qs, cache, block_table, bt_stride, seq_desc, n_seqs, longest, T_, heads, kv_heads, dim, vdim,
+                              block_size, window, sink, gate, ld_gate, channel_gate, out, st);
     }
+    const bool dec = rep <= 16, tiles = !dec || T_ > n_seqs;
     const int dkeys = window_attn_decode_keys(dim, vdim);
     const size_t dsm = std::max((size_t)16 * (dim + 8) * 2 + (size_t)WDEC_WARPS * 2 * dkeys * (dim + vdim + 16) * 2,
                                 (size_t)16 * (dim + 8) * 2 + (size_t)WDEC_WARPS * 16 * (vdim + 2) * 4);

@@ -672,6 +672,48 @@ def test_preparations_read_the_table(cuda):
         assert float(cache[[1, 2, 5, 6, 8]].min()) == 5.0 and float(cache[[1, 2, 5, 6, 8]].max()) == 5.0
 
 
+@pytest.mark.parametrize("H,G,D,V,rd,norm", [(4, 2, 64, 64, 32, 1), (3, 1, 24, 40, 16, 1), (16, 4, 128, 128, 128, 1),
+                                              (2, 2, 48, 8, 0, 1), (5, 5, 16, 16, 16, 0), (40, 20, 128, 128, 64, 1)])
+def test_query_and_key_preparation_bf16(cuda, H, G, D, V, rd, norm):
+    """eight values per thread: norms over the whole projection, turned and unturned pieces, values, places that no token
+    names, a token without a place, sizes whose units exceed a block's"""
+    L, lib = _ops()
+    g = torch.Generator().manual_seed(H)
+    T, HD, GD, GV = 5, H * D, G * D, G * V
+    ld = HD + GD + GV + 8
+    proj = torch.randn(T, ld, generator=g).bfloat16()
+    wq, wk = torch.rand(HD, generator=g) + 0.5, torch.rand(GD, generator=g) + 0.5
+    pos = torch.tensor([0, 3, 40, 999, 70000], dtype=torch.int32)
+    slots = torch.tensor([6, 2, -1, 0, 4], dtype=torch.int32)
+    f = O.frequencies({"dims": rd, "base": 100.0}) if rd else O.frequencies(None)
+    a = pos.double()[:, None] * f[None, :]
+    tab = torch.stack([torch.cos(a), torch.sin(a)], -1).float().contiguous()
+
+    def turn(v):
+        n = f.numel()
+        c, s = torch.cos(a)[:, None, :], torch.sin(a)[:, None, :]
+        return torch.cat([v[..., :n] * c - v[..., n:2 * n] * s, v[..., n:2 * n] * c + v[..., :n] * s, v[..., 2 * n:]], -1)
+
+    q, k = proj[:, :HD].double(), proj[:, HD:HD + GD].double()
+    if norm:
+        q, k = O.rms(q, 1e-5) * wq.double(), O.rms(k, 1e-5) * wk.double()
+    q, k = turn(q.view(T, H, D)) * 0.3, turn(k.view(T, G, D))
+    pd, wqd, wkd, td, sl = (t.to(cuda) for t in (proj, wq, wk, tab, slots))
+    qs = torch.zeros(T, HD, device=cuda)
+    cache = torch.full((8, GD + GV), 5.0, dtype=torch.bfloat16, device=cuda)
+    L.check(lib.b200q_window_attn_prep_tab(pd.data_ptr(), ld, 0, HD, HD + GD, None, H, G, D, V, norm, wqd.data_ptr(),
+                                           wkd.data_ptr(), 1e-5, rd, td.data_ptr() if rd else None, sl.data_ptr(), 0.3,
+                                           qs.data_ptr(), cache.data_ptr(), T, L.DTYPE_BF16, None))
+    torch.cuda.synchronize()
+    assert float((qs.cpu().double().view(T, H, D) - q).abs().max()) < 1e-5
+    for t in range(T):
+        if slots[t] >= 0:
+            row = cache[int(slots[t])].float().cpu()
+            assert float((row[:GD].double() - k[t].reshape(-1)).abs().max()) < 2e-2
+            assert torch.equal(row[GD:], proj[t, HD + GD:HD + GD + GV].float())
+    assert float(cache[[1, 3, 5, 7]].float().min()) == 5.0 and float(cache[[1, 3, 5, 7]].float().max()) == 5.0
+
+
 def test_gated_product_without_biases(cuda):
     """the clamped unit in the product's epilogue with no biases equals the plain form"""
     L, lib = _ops()
