@@ -615,11 +615,11 @@ int b200q_latent_portion_attn(const void* q_dev, int ldq, const float* qa_dev, c
                               const int32_t* seq_desc_dev, int n_seqs, int longest, int heads, int dim, int rot_dim, int vdim,
                               int kv_rank, int block_size, int window, float scale, const float* sink_dev,
                               const void* gate_dev, int ld_gate, void* out_dev, void* stream);
-/* routing of B200Q_FF_MOE_GATED over fp32 router logits [T, E]: s = sigmoid(logits), choice = s + correction; only experts
+/* routing of B200Q_FF_MOE_GATED over fp32 router logits [T, E] (rows of stride ld): s = sigmoid(logits), choice = s + correction; only experts
  * of the keep best of n_groups groups (score: sum of the two largest choices of the group) may be chosen; the top largest
  * choices (ties: lowest index) -> idx, wts = s.  shared 1: every token has one more pair, expert E with weight 1.  Outputs
  * as in b200q_moe_route over E + shared groups and top + shared pairs per token. */
-int b200q_moe_route_gated(const float* logits_dev, const float* correction_dev, int T, int E, int top, int n_groups,
+int b200q_moe_route_gated(const float* logits_dev, int ld, const float* correction_dev, int T, int E, int top, int n_groups,
                           int keep, int shared, int32_t* idx_dev, float* wts_dev, int32_t* group_off_dev,
                           int32_t* perm_tok_dev, int32_t* pair_pos_dev, int32_t* tile_tab_dev, int32_t* n_tiles_dev,
                           void* stream);
@@ -947,15 +947,16 @@ int b200q_model_create(const b200q_model_config* cfg, b200q_model_t* out);
  *   2*ff] their biases in the same order; "out" [W, heads*vdim + ff] = [output projection | down projection]; "out_b"
  *   [1, W] (with a feed-forward).  NP is a multiple of 256 from 1024 used rows up, else of 64.
  * B200Q_ARCH_FIMILORN (cfg.layer_form = B200Q_FORM_SANDWICH, cfg.norm_kind = B200Q_NORM_RMS): per layer "norm1", "norm1b"
- *   (and "norm2", "norm2b" with a feed-forward) [1, W], "step" [1, W] where a pass begins, and
- *   retention: "mix.proj" [roundup64(2*heads*dim + 2*heads*vdim), W] (rows: q, k, v, gate), "mix.decay" [1, heads], "mix.o"
- *   window attention (bare, channel_gate, qk_norm 1, sink): "mix.proj" [roundup64(q + k + v + gate rows), W],
+ *   (and "norm2", "norm2b" with a feed-forward) [1, W], "step" [1, W] where a pass begins, and (roundup: zero rows up to a
+ *   multiple of 64, from 1024 rows up of 256)
+ *   retention: "mix.proj" [roundup(2*heads*dim + 2*heads*vdim), W] (rows: q, k, v, gate), "mix.decay" [1, heads], "mix.o"
+ *   window attention (bare, channel_gate, qk_norm 1, sink): "mix.proj" [roundup(q + k + v + gate rows), W],
  *     "mix.q_norm" [1, heads*dim], "mix.k_norm" [1, kv_heads*dim], "mix.sink" [1, heads], "mix.o"
- *   latent attention (q_rank 0, sink): "mix.down" [roundup64(q rows + kv_rank + rot_dim), W], "mix.kv_norm", "mix.sink",
+ *   latent attention (q_rank 0, sink): "mix.down" [roundup(q rows + kv_rank + rot_dim), W], "mix.kv_norm", "mix.sink",
  *     "mix.uk_t", "mix.uv", "mix.o", optionally "mix.uk" [heads*dim, kv_rank] (the key up-projection as it is: prompt
  *     portions then read expanded keys and values where the sizes allow)
  *   clamped ff: "mlp.gate_up" or "mlp.gate_up_il" [2*ff, W], "mlp.down"
- *   gated experts: "mlp.router" [E, W], "mlp.router_bias" [1, E] (the correction), "mlp.experts_gate_up" [N*2*ff, W],
+ *   gated experts: "mlp.router" [roundup(E), W] (zero rows behind the E), "mlp.router_bias" [1, E] (the correction), "mlp.experts_gate_up" [N*2*ff, W],
  *     "mlp.experts_down" [N*W, ff]; a shared expert as large as the others is expert E of these stacks (N = E + 1), one
  *     of another size has "mlp.shared_gate_up" [2*shared_dim, W] and "mlp.shared_down" [W, shared_dim] (N = E) */
 int b200q_model_create_layered(const b200q_model_config* cfg, const b200q_layer_desc* layers,

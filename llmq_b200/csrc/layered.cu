@@ -233,26 +233,27 @@ struct Widths {
   bool moe = false, shared = false, hf = false, side = false, inject = false, keep_x0 = false;
 };
 int64_t pad64(int64_t v) { return (v + 63) & ~(int64_t)63; }
+// rows of a fused projection: whole 64-wide tiles of the product, from 1024 rows up whole 256-wide ones
+int64_t pad_proj(int64_t v) { return v >= 1024 ? (v + 255) & ~(int64_t)255 : pad64(v); }
 // rows of window attention's fused projection: [q | k | v (own keys and values) | gate number per head (not bare) or gate
-// value per channel], with zero rows up to a multiple of 64
+// value per channel], with zero rows behind (pad_proj)
 int64_t window_proj_rows(const b200q_layer_desc& d) {
-  return pad64((int64_t)d.heads * d.dim + (d.kv_from < 0 ? (int64_t)d.kv_heads * (d.dim + d.vdim) : 0) +
+  return pad_proj((int64_t)d.heads * d.dim + (d.kv_from < 0 ? (int64_t)d.kv_heads * (d.dim + d.vdim) : 0) +
                (d.bare ? 0 : d.heads) + (d.channel_gate ? (int64_t)d.heads * d.vdim : 0));
 }
 // rows of latent attention's fused projection with full-rank queries: [q | latent | shared rotated key | gate number
-// per head (head_gate)], with zero rows up to a multiple of 64
+// per head (head_gate)], with zero rows behind (pad_proj)
 int64_t latent_full_rows(const b200q_layer_desc& d) {
-  return pad64((int64_t)d.heads * (d.dim + d.rot_dim) + d.kv_rank + d.rot_dim + (d.head_gate ? d.heads : 0));
+  return pad_proj((int64_t)d.heads * (d.dim + d.rot_dim) + d.kv_rank + d.rot_dim + (d.head_gate ? d.heads : 0));
 }
-int64_t retention_proj_rows(const b200q_layer_desc& d) { return pad64(2 * (int64_t)d.heads * (d.dim + d.vdim)); }
+int64_t retention_proj_rows(const b200q_layer_desc& d) { return pad_proj(2 * (int64_t)d.heads * (d.dim + d.vdim)); }
 // channels of differential attention's q | k | v (k and v with own keys), and the rows of its part of the fused input
 // projection: those channels, a gate number per head, zero rows
 int64_t diff_channels(const b200q_layer_desc& d) {
   return (int64_t)d.heads * 2 * d.dim + (d.kv_from < 0 ? (int64_t)d.kv_heads * (2 * d.dim + d.vdim) : 0);
 }
 int64_t diff_proj_rows(const b200q_layer_desc& d) {
-  const int64_t n = diff_channels(d) + d.heads;
-  return n >= 1024 ? (n + 255) & ~(int64_t)255 : pad64(n);
+  return pad_proj(diff_channels(d) + d.heads);
 }
 int64_t clamped_ff(const b200q_layer_desc& d) { return d.ff == B200Q_FF_CLAMPED ? d.ff_dim : 0; }
 void sequence_mixer_widths(const b200q_layer_desc& d, int64_t W, Widths& w) {
@@ -338,7 +339,7 @@ Widths widths_of(const b200q_model_config& c, const std::vector<b200q_layered_la
     } else if (d.ff == B200Q_FF_MOE_GATED) {
       const int64_t per = d.top_k + (shared_stacked(d) ? 1 : 0);
       w.moe = true;
-      w.experts = std::max<int64_t>(w.experts, d.n_experts + 1);
+      w.experts = std::max<int64_t>(w.experts, pad_proj(d.n_experts + 1));
       w.pairs = std::max<int64_t>(w.pairs, per);
       w.egu = std::max<int64_t>(w.egu, per * 2 * d.ff_dim);
       w.eact = std::max<int64_t>(w.eact, per * d.ff_dim);
@@ -802,7 +803,7 @@ int layered_bind_weight(b200q_model* m, const char* name, const void* p, int64_t
   }
   if (d.ff == B200Q_FF_MOE_GATED) {
     const int64_t N = d.n_experts + (shared_stacked(d) ? 1 : 0);
-    FIELD("mlp.router", l.router, d.n_experts, W)
+    FIELD("mlp.router", l.router, pad_proj(d.n_experts), W)
     FIELD("mlp.router_bias", l.router_bias, 1, d.n_experts)
     FIELD("mlp.experts_gate_up", l.experts_gate_up, N * 2 * d.ff_dim, W)
     FIELD("mlp.experts_down", l.experts_down, N * W, d.ff_dim)
@@ -1256,9 +1257,11 @@ int layered_forward(b200q_model* m, const b200q_batch* b, void* stream) {
     const b200q_layer_desc& d = l.d;
     const bool stacked = shared_stacked(d);
     const int E = d.n_experts, N = E + (stacked ? 1 : 0), K = d.top_k + (stacked ? 1 : 0), F = d.ff_dim, P = T * K;
-    LIN(y->h2, W, l.router, nullptr, y->rlog, E, E, W, 1);
+    // (long steps take the tensor cores over the padded rows, short ones the dot products of the E real ones)
+    const int ER = (int)pad_proj(E);
+    LIN(y->h2, W, l.router, nullptr, y->rlog, ER, T >= 512 ? ER : E, W, 1);
     TRY(EW, (double)T * E * 4,
-        b200q_moe_route_gated(y->rlog, l.router_bias, T, E, d.top_k, d.n_groups, d.keep_groups, stacked ? 1 : 0, y->idx, y->wts,
+        b200q_moe_route_gated(y->rlog, ER, l.router_bias, T, E, d.top_k, d.n_groups, d.keep_groups, stacked ? 1 : 0, y->idx, y->wts,
                               y->group_off, y->perm_tok, y->pair_pos, y->tile_tab, y->n_tiles, stream));
     const bool sorted = dt == B200Q_DTYPE_BF16 && W % 8 == 0;
     if (sorted) TRY(EW, 2.0 * P * W * es, b200q_gather_rows(y->h2, y->perm_tok, y->esrc, P, W, stream));

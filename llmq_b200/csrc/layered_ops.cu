@@ -290,7 +290,7 @@ __global__ void __launch_bounds__(128) rope_q_kernel(const T* __restrict__ q, in
 // steps 1 and 2 in one for full-rank queries (CTA per token): proj = [q (heads x [dim | rot_dim]) | latent | shared
 // rotated key part].  Pairs (i, i + rot_dims/2) of the first rot_dims entries turn by the step's table.
 template <typename T>
-__global__ void __launch_bounds__(128) latent_prep_tab_kernel(const T* __restrict__ proj, int ldp, int heads, int dim,
+__global__ void __launch_bounds__(256) latent_prep_tab_kernel(const T* __restrict__ proj, int ldp, int heads, int dim,
                                                               int kv_rank, int rot_dim, int rot_dims,
                                                               const float2* __restrict__ table,
                                                               const int32_t* __restrict__ slot_mapping,
@@ -1280,22 +1280,26 @@ __global__ void __launch_bounds__(256) layer_sum_kernel(float* __restrict__ x, c
 }
 
 // greedy sampler over fp32 logits (lowest index wins ties) and the bf16 copy the temperature sampler reads
-__global__ void __launch_bounds__(256) argmax_f32_kernel(const float* __restrict__ logits, int32_t* __restrict__ ids,
-                                                         int V) {
-  __shared__ float bv[256];
-  __shared__ int bi[256];
+constexpr int ARGMAX_THREADS = 1024;
+__global__ void __launch_bounds__(ARGMAX_THREADS) argmax_f32_kernel(const float* __restrict__ logits,
+                                                                    int32_t* __restrict__ ids, int V) {
+  __shared__ float bv[ARGMAX_THREADS];
+  __shared__ int bi[ARGMAX_THREADS];
   const float* z = logits + (long long)blockIdx.x * V;
   float v = -INFINITY;
   int ix = 0x7fffffff;
-  for (int c = threadIdx.x; c < V; c += blockDim.x)
-    if (z[c] > v || (z[c] == v && c < ix)) {
-      v = z[c];
+#pragma unroll 8
+  for (int c = threadIdx.x; c < V; c += ARGMAX_THREADS) {
+    const float x = z[c];
+    if (x > v || (x == v && c < ix)) {
+      v = x;
       ix = c;
     }
+  }
   bv[threadIdx.x] = v;
   bi[threadIdx.x] = ix;
   __syncthreads();
-  for (int o = 128; o > 0; o >>= 1) {
+  for (int o = ARGMAX_THREADS / 2; o > 0; o >>= 1) {
     if (threadIdx.x < o) {
       const float ov = bv[threadIdx.x + o];
       const int oi = bi[threadIdx.x + o];
@@ -1459,7 +1463,7 @@ int b200q_latent_prep_tab(const void* proj, int ldp, int heads, int dim, int kv_
                   "latent_prep: bad argument (heads=%d dim=%d kv_rank=%d rot_dim=%d rot_dims=%d)", heads, dim, kv_rank, rot_dim,
                   rot_dims);
   if (T_ == 0) return B200Q_OK;
-  DISPATCH_T(dtype, (latent_prep_tab_kernel<T><<<T_, 128, (size_t)(rot_dims / 2 + 1) * sizeof(float2), as_stream(stream)>>>(
+  DISPATCH_T(dtype, (latent_prep_tab_kernel<T><<<T_, 256, (size_t)(rot_dims / 2 + 1) * sizeof(float2), as_stream(stream)>>>(
                         (const T*)proj, ldp, heads, dim, kv_rank, rot_dim, rot_dims, (const float2*)table, slot_mapping, w_kvn,
                         qa, (T*)cache, eps)));
   B200Q_LAUNCH_CHECK();
@@ -1721,7 +1725,7 @@ int b200q_layer_sum(float* x, const void* mix, const void* f, const void* expert
 int b200q_argmax_f32(const float* logits, int32_t* ids, int B, int V, void* stream) {
   B200Q_CHECK_ARG(logits && ids && B >= 0 && V > 0, "argmax_f32: bad argument");
   if (B == 0) return B200Q_OK;
-  argmax_f32_kernel<<<B, 256, 0, as_stream(stream)>>>(logits, ids, V);
+  argmax_f32_kernel<<<B, ARGMAX_THREADS, 0, as_stream(stream)>>>(logits, ids, V);
   B200Q_LAUNCH_CHECK();
   return B200Q_OK;
 }

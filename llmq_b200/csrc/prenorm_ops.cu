@@ -209,7 +209,7 @@ __global__ void __launch_bounds__(256) decay_from_logits_kernel(float* __restric
 // chosen scores as they are, and `shared` appends one pair per token for expert E with weight 1.
 constexpr int ROUTE_MAX_GROUPS = 256;
 template <bool GATED>
-__global__ void __launch_bounds__(128) moe_route_grouped_kernel(const float* __restrict__ logits,
+__global__ void __launch_bounds__(128) moe_route_grouped_kernel(const float* __restrict__ logits, int ld,
                                                                 const float* __restrict__ corr, int Tn, int E, int top,
                                                                 int n_groups, int keep, int shared,
                                                                 int32_t* __restrict__ idx, float* __restrict__ wts) {
@@ -217,7 +217,7 @@ __global__ void __launch_bounds__(128) moe_route_grouped_kernel(const float* __r
   const int wi = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * 4 + wi;
   if (t >= Tn) return;
-  const float* z = logits + (long long)t * E;
+  const float* z = logits + (long long)t * ld;
   float mx = -INFINITY, inv = 1.f;
   if (!GATED) {
     for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
@@ -315,27 +315,41 @@ __global__ void __launch_bounds__(1024) moe_plan_part_kernel(const int32_t* __re
   __syncthreads();
   for (int p = threadIdx.x; p < P; p += blockDim.x) atomicAdd(&counts[idx[p]], 1);
   __syncthreads();
-  if (threadIdx.x == 0) {
-    int run = 0;
-    for (int e = 0; e < E; ++e) {
-      offs[e] = run;
-      run += counts[e];
-    }
-    offs[E] = run;
-    if (tile_tab) {
-      int n = 0;
-      for (int e = 0; e < e_gemm; ++e)
-        for (int r = offs[e]; r < offs[e + 1]; r += 128) {
-          tile_tab[4 * n + 0] = e;
-          tile_tab[4 * n + 1] = r;
-          tile_tab[4 * n + 2] = offs[e + 1];
-          tile_tab[4 * n + 3] = 0;
-          ++n;
+  if (threadIdx.x < 32) {  // first pair and first tile of every expert: running sums, 32 experts at a time
+    const int lane = threadIdx.x;
+    int run = 0, tiles = 0;
+    for (int e0 = 0; e0 < E; e0 += 32) {
+      const int e = e0 + lane, c = e < E ? counts[e] : 0, t = e < e_gemm ? (c + 127) / 128 : 0;
+      int cs = c, ts = t;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int cu = __shfl_up_sync(0xffffffffu, cs, o), tu = __shfl_up_sync(0xffffffffu, ts, o);
+        if (lane >= o) {
+          cs += cu;
+          ts += tu;
         }
-      *n_tiles = n;
+      }
+      if (e < E) {
+        offs[e] = run + cs - c;
+        counts[e] = tiles + ts - t;  // from here on: the expert's first tile
+      }
+      run += __shfl_sync(0xffffffffu, cs, 31);
+      tiles += __shfl_sync(0xffffffffu, ts, 31);
+    }
+    if (lane == 0) {
+      offs[E] = run;
+      if (n_tiles) *n_tiles = tiles;
     }
   }
   __syncthreads();
+  if (tile_tab)
+    for (int e = threadIdx.x; e < e_gemm; e += blockDim.x)
+      for (int r = offs[e], n = counts[e]; r < offs[e + 1]; r += 128, ++n) {
+        tile_tab[4 * n + 0] = e;
+        tile_tab[4 * n + 1] = r;
+        tile_tab[4 * n + 2] = offs[e + 1];
+        tile_tab[4 * n + 3] = 0;
+      }
   for (int e = threadIdx.x; e <= E; e += blockDim.x) group_off[e] = offs[e];
   for (int p = threadIdx.x; p < P; p += blockDim.x) {
     const int e = idx[p];
@@ -522,8 +536,8 @@ int b200q_moe_route_grouped(const float* logits, const float* correction, int T_
                   "moe_route_grouped: bad argument (E=%d top=%d groups=%d keep=%d; groups divide E, at most %d groups, "
                   "top fits the kept groups)", E, top, n_groups, keep, ROUTE_MAX_GROUPS);
   if (T_ == 0) return B200Q_OK;
-  moe_route_grouped_kernel<false><<<(T_ + 3) / 4, 128, 0, as_stream(stream)>>>(logits, correction, T_, E, top, n_groups, keep,
-                                                                              0, idx, wts);
+  moe_route_grouped_kernel<false><<<(T_ + 3) / 4, 128, 0, as_stream(stream)>>>(logits, E, correction, T_, E, top, n_groups,
+                                                                              keep, 0, idx, wts);
   B200Q_LAUNCH_CHECK();
   moe_plan_part_kernel<<<1, 1024, (size_t)(3 * E + 1) * sizeof(int32_t), as_stream(stream)>>>(
       idx, T_ * top, top, E, e_gemm, group_off, perm_tok, pair_pos, tile_tab, n_tiles);
@@ -531,19 +545,19 @@ int b200q_moe_route_grouped(const float* logits, const float* correction, int T_
   return B200Q_OK;
 }
 
-int b200q_moe_route_gated(const float* logits, const float* correction, int T_, int E, int top, int n_groups, int keep,
+int b200q_moe_route_gated(const float* logits, int ld, const float* correction, int T_, int E, int top, int n_groups, int keep,
                           int shared, int32_t* idx, float* wts, int32_t* group_off, int32_t* perm_tok, int32_t* pair_pos,
                           int32_t* tile_tab, int32_t* n_tiles, void* stream) {
   B200Q_CHECK_ARG(!tile_tab == !n_tiles, "moe_route_gated: tile_tab and n_tiles go together");
-  B200Q_CHECK_ARG(logits && correction && idx && wts && group_off && perm_tok && pair_pos && T_ >= 0 && E > 0 && E + shared < 4096 &&
+  B200Q_CHECK_ARG(logits && correction && idx && wts && group_off && perm_tok && pair_pos && T_ >= 0 && E > 0 && ld >= E && E + shared < 4096 &&
                       top > 0 && top <= 32 && n_groups > 0 && n_groups <= ROUTE_MAX_GROUPS && E % n_groups == 0 && keep > 0 &&
                       keep <= n_groups && top <= keep * (E / n_groups) && (shared == 0 || shared == 1),
                   "moe_route_gated: bad argument (E=%d top=%d groups=%d keep=%d; groups divide E, at most %d groups, top fits "
                   "the kept groups)", E, top, n_groups, keep, ROUTE_MAX_GROUPS);
   if (T_ == 0) return B200Q_OK;
   const int per = top + shared, n = E + shared;
-  moe_route_grouped_kernel<true><<<(T_ + 3) / 4, 128, 0, as_stream(stream)>>>(logits, correction, T_, E, top, n_groups, keep,
-                                                                             shared, idx, wts);
+  moe_route_grouped_kernel<true><<<(T_ + 3) / 4, 128, 0, as_stream(stream)>>>(logits, ld, correction, T_, E, top, n_groups,
+                                                                             keep, shared, idx, wts);
   B200Q_LAUNCH_CHECK();
   moe_plan_part_kernel<<<1, 1024, (size_t)(3 * n + 1) * sizeof(int32_t), as_stream(stream)>>>(
       idx, T_ * per, per, n, n, group_off, perm_tok, pair_pos, tile_tab, n_tiles);

@@ -61,16 +61,31 @@ __global__ void __launch_bounds__(RET_THREADS) retention_decode_kernel(
   const float2* cs = table + t * half;
   float *qs = sm, *ks = sm + dim, *part = sm + 2 * dim;
   const float kmul = 1.f / sqrtf((float)dim), lam = decay[h];
+  const int nc = vdim / V, groups = nc < RET_THREADS ? RET_THREADS / nc : 1;
+  const int grp = nc < RET_THREADS ? tid / nc : 0, cv0 = nc < RET_THREADS ? tid % nc : tid;
+  float* st = state + (long long)s.slot * slot_stride + (long long)h * dim * vdim;
+  float S[RET_ROWS][V];
+  auto fetch = [&](int d0, int c) {
+#pragma unroll
+    for (int r = 0; r < RET_ROWS; ++r) {
+      const int d = d0 + r * groups;
+      const bool on = d < dim && s.pos0 > 0;  // a sequence that starts here starts from zeros whatever the slot holds
+      if constexpr (V == 4) {
+        const float4 f = on ? *reinterpret_cast<const float4*>(st + (long long)d * vdim + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        S[r][0] = f.x; S[r][1] = f.y; S[r][2] = f.z; S[r][3] = f.w;
+      } else {
+        S[r][0] = on ? st[(long long)d * vdim + c] : 0.f;
+      }
+    }
+  };
+  if (grp < groups && cv0 < nc) fetch(grp, cv0 * V);  // on its way while the vectors are turned
   for (int d = tid; d < dim; d += RET_THREADS) {
     qs[d] = turned(pr + h * dim, d, half, cs);
     ks[d] = turned(pr + HD + h * dim, d, half, cs) * kmul;
   }
   __syncthreads();
-  const int nc = vdim / V, groups = nc < RET_THREADS ? RET_THREADS / nc : 1;
-  const int grp = nc < RET_THREADS ? tid / nc : 0;
-  float* st = state + (long long)s.slot * slot_stride + (long long)h * dim * vdim;
   if (grp < groups)
-    for (int cv = nc < RET_THREADS ? tid % nc : tid; cv < nc; cv += RET_THREADS) {
+    for (int cv = cv0; cv < nc; cv += RET_THREADS) {
       const int c = cv * V;
       float v[V], o[V];
 #pragma unroll
@@ -79,18 +94,7 @@ __global__ void __launch_bounds__(RET_THREADS) retention_decode_kernel(
         o[i] = 0.f;
       }
       for (int d0 = grp; d0 < dim; d0 += groups * RET_ROWS) {
-        float S[RET_ROWS][V];
-#pragma unroll
-        for (int r = 0; r < RET_ROWS; ++r) {
-          const int d = d0 + r * groups;
-          const bool on = d < dim && s.pos0 > 0;  // a sequence that starts here starts from zeros whatever the slot holds
-          if constexpr (V == 4) {
-            const float4 f = on ? *reinterpret_cast<const float4*>(st + (long long)d * vdim + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-            S[r][0] = f.x; S[r][1] = f.y; S[r][2] = f.z; S[r][3] = f.w;
-          } else {
-            S[r][0] = on ? st[(long long)d * vdim + c] : 0.f;
-          }
-        }
+        if (d0 != grp || cv != cv0) fetch(d0, c);
 #pragma unroll
         for (int r = 0; r < RET_ROWS; ++r) {
           const int d = d0 + r * groups;

@@ -188,16 +188,15 @@ __device__ __forceinline__ void close_value(const CloseSource& s, long long t, i
 
 // CTA per row; rows of up to 256 * V * CLOSE_ROWS values stay in registers between y's norm, the sum and x's norm, the
 // rest of a longer row is worked out again
-constexpr int CLOSE_ROWS = 4;
-template <typename TY, typename T, int V>
-__global__ void __launch_bounds__(256) sandwich_close_kernel(float* __restrict__ x, CloseSource s,
+template <typename TY, typename T, int V, int CLOSE_ROWS>
+__global__ void __launch_bounds__(256, CLOSE_ROWS == 2 ? 4 : 2) sandwich_close_kernel(float* __restrict__ x, CloseSource s,
                                                              const float* __restrict__ post_w,
                                                              const float* __restrict__ next_w, T* __restrict__ out, int W,
                                                              float eps) {
   __shared__ float red[32];
   const long long t = blockIdx.x;
   float* xr = x + t * W;
-  float v[CLOSE_ROWS][4];
+  float v[CLOSE_ROWS][4], xk[CLOSE_ROWS][4];
   float ss = 0.f;
   auto sq = [&](const float (&a)[4]) {
 #pragma unroll
@@ -208,8 +207,12 @@ __global__ void __launch_bounds__(256) sandwich_close_kernel(float* __restrict__
   for (int q = 0; q < CLOSE_ROWS; ++q)
     if (c0 + q * step < W) {
       close_value<TY, T, V>(s, t, W, c0 + q * step, v[q]);
-      sq(v[q]);
+      if (V == 4) ld4(xr + c0 + q * step, xk[q]);  // on its way while y's norm is worked out
+      else xk[q][0] = xr[c0 + q * step];
     }
+#pragma unroll
+  for (int q = 0; q < CLOSE_ROWS; ++q)
+    if (c0 + q * step < W) sq(v[q]);
   for (int c = c0 + CLOSE_ROWS * step; c < W; c += step) {
     float a[4];
     close_value<TY, T, V>(s, t, W, c, a);
@@ -217,15 +220,10 @@ __global__ void __launch_bounds__(256) sandwich_close_kernel(float* __restrict__
   }
   const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)W + eps);
   ss = 0.f;
-  auto add = [&](int c, float (&a)[4]) {  // a: y's value, then x's new one
-    float xv[4], w[4];
-    if (V == 4) {
-      ld4(xr + c, xv);
-      ld4(post_w + c, w);
-    } else {
-      xv[0] = xr[c];
-      w[0] = post_w[c];
-    }
+  auto add = [&](int c, float (&a)[4], const float (&xv)[4]) {  // a: y's value, then x's new one
+    float w[4];
+    if (V == 4) ld4(post_w + c, w);
+    else w[0] = post_w[c];
 #pragma unroll
     for (int i = 0; i < V; ++i) a[i] = fmaf(a[i] * inv, w[i], xv[i]);
     if (V == 4) st4(xr + c, a);
@@ -234,11 +232,14 @@ __global__ void __launch_bounds__(256) sandwich_close_kernel(float* __restrict__
   };
 #pragma unroll
   for (int q = 0; q < CLOSE_ROWS; ++q)
-    if (c0 + q * step < W) add(c0 + q * step, v[q]);
+    if (c0 + q * step < W) add(c0 + q * step, v[q], xk[q]);
   for (int c = c0 + CLOSE_ROWS * step; c < W; c += step) {
     float a[4];
+    float xv[4];
     close_value<TY, T, V>(s, t, W, c, a);
-    add(c, a);
+    if (V == 4) ld4(xr + c, xv);
+    else xv[0] = xr[c];
+    add(c, a, xv);
   }
   if (!next_w) return;
   const float inv2 = 1.f / sqrtf(block_sum(ss, red) / (float)W + eps);
@@ -429,8 +430,13 @@ int b200q_sandwich_close(float* x, const void* y, int y_f32, int splits, const i
                                   reinterpret_cast<uintptr_t>(y2) | reinterpret_cast<uintptr_t>(post_w) |
                                   reinterpret_cast<uintptr_t>(next_w) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
   cudaStream_t st = as_stream(stream);
-#define CLOSE(TY, V)                                                                                                      \
-  DISPATCH_T(dtype, (sandwich_close_kernel<TY, T, V><<<T_, 256, 0, st>>>(x, s, post_w, next_w, (T*)out, W, eps)))
+#define CLOSE(TY, V)                                                                                                       \
+  do {                                                                                                                    \
+    if (W <= 256 * V * 2)                                                                                                 \
+      DISPATCH_T(dtype, (sandwich_close_kernel<TY, T, V, 2><<<T_, 256, 0, st>>>(x, s, post_w, next_w, (T*)out, W, eps))); \
+    else                                                                                                                  \
+      DISPATCH_T(dtype, (sandwich_close_kernel<TY, T, V, 4><<<T_, 256, 0, st>>>(x, s, post_w, next_w, (T*)out, W, eps))); \
+  } while (0)
   if (y_f32) {
     if (v4) CLOSE(float, 4);
     else CLOSE(float, 1);

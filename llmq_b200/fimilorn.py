@@ -256,7 +256,7 @@ def engine_weights(spec: FimilornSpec, sd: Dict[str, torch.Tensor]) -> Iterable[
     (bound in the model's dtype); 1-D results are vectors and constants (bound as fp32 rows).  Runs of the same
     checkpoint layer yield the SAME tensor objects, which the model uploads once.  Fusions: the projections that read a
     mixer's input become one matrix with zero rows up to a multiple of 64 (retention and attention: q, k, v, gate;
-    latent attention: q, the latent, the shared rotated key); each head's key up-projection is stored transposed too (single
+    latent attention: q, the latent, the shared rotated key; the router alone); each head's key up-projection is stored transposed too (single
     tokens carry the query into the latent space); gate and up of the dense unit are stacked (interleaved in blocks of 128 rows
     when ff is a multiple of 128); the experts' matrices are stacked, a shared expert of their size as one more."""
     yield "embed", sd["embed"]
@@ -308,7 +308,7 @@ def _layer_weights(ly: FimilornLayer, sd) -> Iterable[Tuple[str, torch.Tensor]]:
             yield "mlp.gate_up", torch.cat([sd[f + "gate"], sd[f + "up"]], 0)
         yield "mlp.down", sd[f + "down"]
         return
-    yield "mlp.router", sd[f + "router"]
+    yield "mlp.router", _pad_rows(sd[f + "router"])
     yield "mlp.router_bias", sd[f + "correction"].reshape(-1)
     stack = [f"{f}e{e}." for e in range(ly.n_experts)]
     if ly.shared_ff and ly.shared_ff == ly.ff_dim:

@@ -238,8 +238,9 @@ class KabavikSpec:
 
 
 # ---- checkpoint names -> engine names --------------------------------------------------------------
-def _pad_rows(t: torch.Tensor, mult: int = 64) -> torch.Tensor:
-    pad = -t.shape[0] % mult
+def _pad_rows(t: torch.Tensor) -> torch.Tensor:
+    """zero rows behind a fused projection: whole 64-wide tiles of the product, from 1024 rows up whole 256-wide ones"""
+    pad = -t.shape[0] % (256 if t.shape[0] >= 1024 else 64)
     return torch.cat([t, t.new_zeros((pad,) + tuple(t.shape[1:]))], 0) if pad else t
 
 

@@ -527,8 +527,8 @@ def test_routing_by_groups(cuda):
             ints = lambda n: torch.full((n,), -1, dtype=torch.int32, device=cuda)
             idx, off, perm, pair, tab, nt = ints(T * K), ints(N + 1), ints(T * K), ints(T * K), ints((T * K // 128 + N + 1) * 4), ints(4)
             wts = torch.zeros(T * K, device=cuda)
-            zd, cd = z.to(cuda), corr.to(cuda)
-            L.check(lib.b200q_moe_route_gated(zd.data_ptr(), cd.data_ptr(), T, E, top, n_groups, keep, shared, idx.data_ptr(),
+            zd, cd = torch.cat([z, torch.full((T, 3), 50.0)], 1).to(cuda), corr.to(cuda)   # (rows are wider than E)
+            L.check(lib.b200q_moe_route_gated(zd.data_ptr(), E + 3, cd.data_ptr(), T, E, top, n_groups, keep, shared, idx.data_ptr(),
                                               wts.data_ptr(), off.data_ptr(), perm.data_ptr(), pair.data_ptr(), tab.data_ptr(),
                                               nt.data_ptr(), None))
             torch.cuda.synchronize()

@@ -135,6 +135,8 @@ def test_engine_weights_shapes_fusions_and_sharing():
     assert ew["layers.2.mlp.experts_gate_up"].shape == (6 * 48, W) and ew["layers.2.mlp.shared_gate_up"].shape == (112, W)
     assert "layers.3.norm2" not in ew and "layers.3.mlp.router" not in ew
     assert "layers.10.mlp.shared_gate_up" not in ew
+    router = ew["layers.1.mlp.router"]
+    assert router.shape == (64, W) and torch.equal(router[:12], sd["l1.mlp.router"]) and float(router[12:].abs().max()) == 0.0
     # runs of one layer share their tensors; every pass has its own step vector
     for n in ("mix.down", "mlp.experts_gate_up", "norm1b"):
         assert ew[f"layers.1.{n}"] is ew[f"layers.4.{n}"] is ew[f"layers.7.{n}"]
@@ -231,6 +233,6 @@ def test_op_arguments_are_checked_before_any_launch():
     assert lib.b200q_retention_scratch_floats(3, 8, 16) == 3 * 48
     assert lib.b200q_retention(None, 0, 1, 8, 8, 0, None, None, None, 0, None, None, 1, 1, 1e-5, None, None, 1, 0, None) == -1
     assert b"retention" in lib.b200q_last_error()
-    assert lib.b200q_moe_route_gated(None, None, 1, 6, 2, 4, 1, 0, *([None] * 8)) == -1
+    assert lib.b200q_moe_route_gated(None, 6, None, 1, 6, 2, 4, 1, 0, *([None] * 8)) == -1
     assert lib.b200q_sandwich_close(None, None, 0, 1, None, None, 0, None, None, None, None, 1, 8, 1e-5, 0, None) == -1
     assert lib.b200q_pass_begin(None, None, None, None, None, None, 1, 8, 1e-5, 0, None) == -1
