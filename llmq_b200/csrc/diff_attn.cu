@@ -364,16 +364,6 @@ __global__ void __launch_bounds__(256) diff_attn_kernel(DiffAttn a) {
   }
 }
 
-// ---- bounded wait on an mbarrier: false when it ran out (about two seconds), so that a kernel can give up ----
-__device__ __forceinline__ bool mbar_wait_limited(uint64_t* bar, uint32_t parity) {
-  const long long t0 = clock64();
-  for (int i = 0; i < (1 << 26); ++i) {
-    if (mbar_try_wait(bar, parity)) return true;
-    if (clock64() - t0 > 4000000000ll) break;
-  }
-  return false;
-}
-
 constexpr float DATT_NEG = -1e30f;  // finite floor of the running maximum: exp2(masked - floor) = 0, never NaN
 constexpr int DATT_PAGE = 16;       // cached rows of a page (= block size)
 
@@ -800,12 +790,8 @@ __global__ void __launch_bounds__(128) diff_attn_decode_kernel(DiffAttn a) {
   }
 }
 
-}  // namespace b200q
-
-using namespace b200q;
-
 // one flag in mapped host memory for the process: a kernel whose wait ran out sets it, the host reads it without a copy
-static int* wait_flag(int** dev) {
+int* wait_flag(int** dev) {
   static int *host = nullptr, *device = nullptr;
   if (!host) {
     if (cudaHostAlloc((void**)&host, 64, cudaHostAllocMapped) != cudaSuccess) return nullptr;
@@ -815,6 +801,10 @@ static int* wait_flag(int** dev) {
   if (dev) *dev = device;
   return host;
 }
+
+}  // namespace b200q
+
+using namespace b200q;
 
 // most tokens of a portion: what the caller says, or what a step of T tokens leaves for one of n_seqs sequences
 static int longest_portion(int max_portion, int n_seqs, int T) {

@@ -34,6 +34,17 @@ __device__ __forceinline__ float sigmoidf_(float x) { return 1.f / (1.f + expf(-
 __device__ __forceinline__ float siluf_(float x) { return x / (1.f + expf(-x)); }
 __device__ __forceinline__ float softplusf_(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 
+// ---- bounded wait on an mbarrier: false when it ran out (about two seconds), so that a kernel can give up ----
+__device__ __forceinline__ bool mbar_wait_limited(uint64_t* bar, uint32_t parity) {
+  const long long t0 = clock64();
+  for (int i = 0; i < (1 << 26); ++i) {
+    if (mbar_try_wait(bar, parity)) return true;
+    if (clock64() - t0 > 4000000000ll) break;
+  }
+  return false;
+}
+int* wait_flag(int** dev);  // where such a kernel says so (diff_attn.cu): host and device address of one int
+
 static inline int grid_for(long long total, int block = 256) {
   long long g = (total + block - 1) / block;
   return (int)(g < 1 ? 1 : (g > 148 * 16 ? 148 * 16 : g));
@@ -43,6 +54,11 @@ bool portion_attn_gqa_ok(const float* qs, const void* cache, const void* out, in
 int portion_attn_gqa(const float* qs, const void* cache, const int32_t* block_table, int bt_stride, const int32_t* seq_desc,
                      int n_seqs, int longest, int T, int heads, int kv_heads, int dim, int vdim, int block_size, int window,
                      const float* sink, const void* gate, int ld_gate, int channel_gate, void* out, cudaStream_t st);
+// ... and attention in the latent space (behind b200q_latent_attn_sink)
+bool latent_tokens_ok(const float* qa, const void* cache, const void* out, int R, int P, int block_size);
+int latent_tokens(const float* qa, const void* cache, const int32_t* block_table, int bt_stride, const int32_t* row_seq,
+                  const int32_t* positions, int T, int heads, int R, int P, int block_size, int window, float scale,
+                  const float* sink, const void* gate, int ld_gate, void* out, cudaStream_t st);
 
 static inline bool is_dtype(int d) { return d == B200Q_DTYPE_BF16 || d == B200Q_DTYPE_F32; }
 

@@ -1524,6 +1524,9 @@ int b200q_latent_attn_sink(const float* qa, const void* cache, const int32_t* bl
     return v ? v[0] : '2';
   }();
   const bool use_mma = mma_mode != '0';
+  if (mma_mode == '2' && dtype == B200Q_DTYPE_BF16 && latent_tokens_ok(qa, cache, out, kv_rank, rot_dim, block_size))
+    return latent_tokens(qa, cache, block_table, bt_stride, row_seq, positions, T_, heads, kv_rank, rot_dim, block_size, window,
+                         scale, sink, gate, ld_gate, out, as_stream(stream));
   if (use_mma && dtype == B200Q_DTYPE_BF16 && kv_rank % 64 == 0 && kv_rank <= 512 && RP % 16 == 0 &&
       (reinterpret_cast<uintptr_t>(cache) & 15) == 0 && (reinterpret_cast<uintptr_t>(out) & 3) == 0) {
     const int LDS = RP + 8;

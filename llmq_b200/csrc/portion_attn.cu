@@ -6,7 +6,7 @@
 //                             expanded row many times, so expanding it once costs less than carrying every query into the
 //                             latent space (which single tokens do): per score dim + rot_dim + vdim products instead of
 //                             2 kv_rank + rot_dim.
-// Single tokens of grouped-query attention: one CTA per (sequence, key head), below.
+// Single tokens: one CTA per (sequence, key head), and per (token, 16 or 32 heads) in the latent space, below.
 // Scores, softmax state and accumulators are fp32; queries and weights are rounded to bf16 as the products see them.
 #include <stdlib.h>
 
@@ -495,6 +495,239 @@ __global__ void __launch_bounds__(256) token_attn_kernel(const PortionAttn a) {
   }
 }
 
+// ------------------------------------------------------------------------------------------------
+// latent attention in the latent space (single tokens, and portions that are not worth expanding): one CTA of 8 warps per
+// (token, MT * 16 heads).  A cached row [latent | rotated part] serves all of the CTA's heads as key and, its latent, as value.
+// Chunks of CH = 64 / MT keys pass through a ring of STG stages, a row = one bulk copy (the warps ask
+// for an eighth of a chunk each: a warp's lanes issue their copies one after the other).  Every warp scores one 16 x 8 tile of (heads, keys) over all
+// kv_rank + rot_dim dimensions (queries as bf16 high and low parts, read from shared memory), the scores meet in shared
+// memory, and every warp accumulates kv_rank / 8 of the latent dimensions.  Chunks start at the token's first visible key, so
+// its arithmetic does not depend on how the prompt was cut.  Needs kv_rank a multiple of 128 up to 512.
+// ------------------------------------------------------------------------------------------------
+struct LatentTokens {
+  const float* qa;    // [T, heads, RP]
+  const bf16* cache;  // paged rows of RP elements
+  const int32_t *block_table, *row_seq, *positions;
+  const float* sink;
+  const bf16* gate;
+  bf16* out;  // [T, heads, R]
+  int* failed;  // set when a bounded wait runs out
+  float scale;  // of the scores, in base 2
+  int bt_stride, heads, R, RP, bs_shift, window, ld_gate;
+};
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+template <int MT, int NT>  // NT: 8-wide tiles of latent dimensions per warp
+__global__ void __launch_bounds__(256, 1) latent_token_kernel(const LatentTokens a) {
+  constexpr int CH = 64 / MT, STG = MT == 1 ? 2 : 3, SLD = CH + 4, NK = CH / 8;
+  extern __shared__ __align__(128) uint8_t smraw[];
+  __shared__ __align__(8) uint64_t full[STG];
+  const int LDS = a.RP + 8;  // padded rows: ldmatrix rows fall on different banks
+  bf16* ring = reinterpret_cast<bf16*>(smraw);                   // [STG][CH][LDS]
+  bf16* qhi = ring + STG * CH * LDS;                             // [MT*16][LDS]
+  bf16* qlo = qhi + MT * 16 * LDS;                               // [MT*16][LDS]
+  float* sc = reinterpret_cast<float*>(qlo + MT * 16 * LDS);     // [MT*16][SLD]
+  const int t = blockIdx.x, h0 = blockIdx.y * MT * 16;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gq = lane >> 2, q4 = lane & 3;
+  const int p = a.positions[t], lo = a.window > 0 ? max(0, p - a.window + 1) : 0;
+  const int nchunks = (p - lo) / CH + 1;
+  const int32_t* bt = a.block_table + (long long)a.row_seq[t] * a.bt_stride;
+  const int page_mask = (1 << a.bs_shift) - 1;
+  // lanes l < CH / 8 of warp w ask for key w * CH / 8 + l of a chunk; row_next: its cache row in the next chunk to be asked for
+  const int key_of = warp * (CH / 8) + (lane & (CH / 8 - 1));
+  int row_next = 0;
+  auto look_up = [&](int c) {
+    const int pos = min(lo + c * CH + key_of, p);
+    row_next = (bt[pos >> a.bs_shift] << a.bs_shift) + (pos & page_mask);
+  };
+  auto load_chunk = [&](int c) {
+    const int stage = c % STG, n = min(CH, p + 1 - (lo + c * CH));
+    if (tid == 0) mbar_expect_tx(full + stage, (uint32_t)(n * a.RP * 2));  // (copies that land first wait for it)
+    if (lane < CH / 8 && key_of < n)
+      tma_bulk_g2s(ring + (stage * CH + key_of) * LDS, a.cache + (long long)row_next * a.RP, (uint32_t)(a.RP * 2), full + stage);
+    __syncwarp();
+  };
+  look_up(0);
+  if (tid == 0) {
+#pragma unroll
+    for (int i = 0; i < STG; ++i) mbar_init(full + i, 1);
+    mbar_fence_init();
+  }
+  __syncthreads();  // the barriers are there
+#pragma unroll
+  for (int c = 0; c < STG - 1; ++c)
+    if (c < nchunks) {
+      load_chunk(c);
+      if (c + 1 < nchunks) look_up(c + 1);
+    }
+  for (int e = tid; e < MT * 16 * (a.RP / 4); e += 256) {
+    const int r = e / (a.RP / 4), d = (e % (a.RP / 4)) * 4;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (h0 + r < a.heads) v = *reinterpret_cast<const float4*>(a.qa + ((long long)t * a.heads + h0 + r) * a.RP + d);
+    const float x[4] = {v.x * a.scale, v.y * a.scale, v.z * a.scale, v.w * a.scale};
+    const uint32_t w0 = pack_bf16x2(x[0], x[1]), w1 = pack_bf16x2(x[2], x[3]);
+    *reinterpret_cast<uint2*>(qhi + r * LDS + d) = make_uint2(w0, w1);
+    *reinterpret_cast<uint2*>(qlo + r * LDS + d) =
+        make_uint2(pack_bf16x2(x[0] - bf16_lo(w0), x[1] - bf16_hi(w0)), pack_bf16x2(x[2] - bf16_lo(w1), x[3] - bf16_hi(w1)));
+  }
+  const int mt = warp / NK, nk = warp % NK;  // the score tile of this warp
+  const uint32_t a_off = (uint32_t)(((mt * 16 + (lane & 15)) * LDS + (lane >> 4) * 8) * 2);
+  const uint32_t qhi_s = smem_u32(qhi) + a_off, qlo_s = smem_u32(qlo) + a_off;
+  const uint32_t k_off = (uint32_t)(((nk * 8 + (lane & 7)) * LDS + 8 * (lane >> 3)) * 2);  // 8 keys x 32 dimensions
+  const int dim_w = warp * NT * 8;
+  float m_[MT][2], l_[MT][2], o[MT][NT][4];
+#pragma unroll
+  for (int m = 0; m < MT; ++m) {
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      const int h = h0 + m * 16 + gq + 8 * r;
+      const bool on = a.sink && h < a.heads;  // every thread holds its rows' whole sums: the sink's 1 belongs to each
+      m_[m][r] = on ? a.sink[h] * 1.4426950408889634f : -INFINITY;
+      l_[m][r] = on ? 1.f : 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < NT; ++i) o[m][i][0] = o[m][i][1] = o[m][i][2] = o[m][i][3] = 0.f;
+  }
+  for (int c = 0; c < nchunks; ++c) {
+    const int n = min(CH, p + 1 - (lo + c * CH));
+    bool ok = mbar_wait_limited(full + c % STG, (uint32_t)(c / STG) & 1u);
+    if (n < CH)  // rows behind the last key: their weights are zeros, their values must not be NaNs
+      for (int e = tid; e < (CH - n) * (a.R / 8); e += 256)
+        st_v4(ring + ((c % STG) * CH + n + e / (a.R / 8)) * LDS + (e % (a.R / 8)) * 8, make_uint4(0, 0, 0, 0));
+    ok = __syncthreads_and(ok);  // chunk c (and, first time, the queries) is there; chunk c - 1 and its scores are done with
+    if (!ok) {  // give up: let the copies already on their way land first
+      if (tid == 0) {
+        for (int i = c + 1; i < c + STG - 1 && i < nchunks; ++i) mbar_wait_limited(full + i % STG, (uint32_t)(i / STG) & 1u);
+        *(volatile int*)a.failed = 1;
+      }
+      return;
+    }
+    if (c + STG - 1 < nchunks) {
+      load_chunk(c + STG - 1);
+      if (c + STG < nchunks) look_up(c + STG);
+    }
+    const uint32_t kb_s = smem_u32(ring + (c % STG) * CH * LDS);
+    {
+      float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f}, u0[4] = {0.f, 0.f, 0.f, 0.f}, u1[4] = {0.f, 0.f, 0.f, 0.f};
+      int d = 0;
+#pragma unroll 3
+      for (; d + 32 <= a.RP; d += 32) {
+        uint32_t b0, b1, b2, b3, h0_, h1, h2, h3, g0, g1, g2, g3;
+        ldsm_x4(kb_s + k_off + d * 2, b0, b1, b2, b3);
+        ldsm_x4(qhi_s + d * 2, h0_, h1, h2, h3);
+        ldsm_x4(qlo_s + d * 2, g0, g1, g2, g3);
+        mma_bf16_16816(s0, h0_, h1, h2, h3, b0, b1);
+        mma_bf16_16816(u0, g0, g1, g2, g3, b0, b1);
+        ldsm_x4(qhi_s + d * 2 + 32, h0_, h1, h2, h3);
+        ldsm_x4(qlo_s + d * 2 + 32, g0, g1, g2, g3);
+        mma_bf16_16816(s1, h0_, h1, h2, h3, b2, b3);
+        mma_bf16_16816(u1, g0, g1, g2, g3, b2, b3);
+      }
+      if (d < a.RP) {  // 16 dimensions left
+        uint32_t b0, b1, b2, b3, h0_, h1, h2, h3;
+        ldsm_x4(kb_s + k_off + d * 2 - 32, b0, b1, b2, b3);  // (from 16 before: the last 32 of the row)
+        ldsm_x4(qhi_s + d * 2, h0_, h1, h2, h3);
+        mma_bf16_16816(s0, h0_, h1, h2, h3, b2, b3);
+        ldsm_x4(qlo_s + d * 2, h0_, h1, h2, h3);
+        mma_bf16_16816(u0, h0_, h1, h2, h3, b2, b3);
+      }
+      float* dst = sc + (mt * 16 + gq) * SLD + nk * 8 + 2 * q4;
+      *reinterpret_cast<float2*>(dst) = make_float2((s0[0] + s1[0]) + (u0[0] + u1[0]), (s0[1] + s1[1]) + (u0[1] + u1[1]));
+      *reinterpret_cast<float2*>(dst + 8 * SLD) = make_float2((s0[2] + s1[2]) + (u0[2] + u1[2]), (s0[3] + s1[3]) + (u0[3] + u1[3]));
+    }
+    __syncthreads();
+    uint32_t pk[MT][NK * 2];
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {
+      float corr[2];
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        const float* src = sc + (m * 16 + gq + 8 * r) * SLD + 2 * q4;
+        float v[NK * 2], mx = -INFINITY;
+#pragma unroll
+        for (int k = 0; k < NK; ++k) {
+          const float2 x = *reinterpret_cast<const float2*>(src + 8 * k);
+          v[2 * k] = x.x;
+          v[2 * k + 1] = x.y;
+        }
+        if (n < CH) {
+#pragma unroll
+          for (int k = 0; k < NK * 2; ++k)
+            if ((k >> 1) * 8 + 2 * q4 + (k & 1) >= n) v[k] = -INFINITY;
+        }
+#pragma unroll
+        for (int k = 0; k < NK * 2; ++k) mx = fmaxf(mx, v[k]);
+        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+        const float mn = fmaxf(m_[m][r], mx);
+        corr[r] = ex2(m_[m][r] - mn);
+        m_[m][r] = mn;
+        float ps = 0.f;
+#pragma unroll
+        for (int k = 0; k < NK; ++k) {
+          // rounded to what the value product sees (bf16), so that a row's weights still add up to one
+          const uint32_t w = pack_bf16x2(ex2(v[2 * k] - mn), ex2(v[2 * k + 1] - mn));
+          ps += bf16_lo(w) + bf16_hi(w);
+          pk[m][(k >> 1) * 4 + (k & 1) * 2 + r] = w;
+        }
+        ps += __shfl_xor_sync(0xffffffffu, ps, 1);
+        ps += __shfl_xor_sync(0xffffffffu, ps, 2);
+        l_[m][r] = l_[m][r] * corr[r] + ps;
+      }
+      if (__any_sync(0xffffffffu, corr[0] != 1.f || corr[1] != 1.f)) {
+#pragma unroll
+        for (int i = 0; i < NT; ++i) {
+          o[m][i][0] *= corr[0];
+          o[m][i][1] *= corr[0];
+          o[m][i][2] *= corr[1];
+          o[m][i][3] *= corr[1];
+        }
+      }
+    }
+#pragma unroll
+    for (int kk = 0; kk < CH / 16; ++kk) {
+      const int key = kk * 16 + ((lane >> 3) & 1) * 8 + (lane & 7);
+      const uint32_t v_row = kb_s + (uint32_t)((key * LDS + dim_w + 8 * (lane >> 4)) * 2);
+#pragma unroll
+      for (int nd = 0; nd < NT / 2; ++nd) {
+        uint32_t b0, b1, b2, b3;
+        ldsm_x4_t(v_row + nd * 32, b0, b1, b2, b3);
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+          mma_bf16_16816(o[m][2 * nd], pk[m][4 * kk], pk[m][4 * kk + 1], pk[m][4 * kk + 2], pk[m][4 * kk + 3], b0, b1);
+          mma_bf16_16816(o[m][2 * nd + 1], pk[m][4 * kk], pk[m][4 * kk + 1], pk[m][4 * kk + 2], pk[m][4 * kk + 3], b2, b3);
+        }
+      }
+    }
+  }
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      const int h = h0 + m * 16 + gq + 8 * r;
+      if (h >= a.heads) continue;
+      const float inv = (a.gate ? sigmoidf_(__bfloat162float(a.gate[(long long)t * a.ld_gate + h])) : 1.f) / l_[m][r];
+      bf16* orow = a.out + ((long long)t * a.heads + h) * a.R + dim_w + 2 * q4;
+#pragma unroll
+      for (int i = 0; i < NT; ++i)
+        *reinterpret_cast<uint32_t*>(orow + i * 8) = pack_bf16x2(o[m][i][2 * r] * inv, o[m][i][2 * r + 1] * inv);
+    }
+}
+
+template <int MT, int NT>
+static int launch_latent_tokens(const LatentTokens& a, int T, cudaStream_t st) {
+  constexpr int CH = 64 / MT, STG = MT == 1 ? 2 : 3;
+  const int smem = ((STG * CH + 2 * MT * 16) * (a.RP + 8)) * 2 + MT * 16 * (CH + 4) * 4;
+  auto kern = latent_token_kernel<MT, NT>;
+  B200Q_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+  kern<<<dim3(T, (a.heads + MT * 16 - 1) / (MT * 16)), 256, smem, st>>>(a);
+  B200Q_LAUNCH_CHECK();
+  return B200Q_OK;
+}
+
 static int shift_of(int block_size) {  // -1: not a power of two
   int s = 0;
   while ((1 << s) < block_size) ++s;
@@ -536,6 +769,35 @@ static bool portion_attn_on() {  // B200Q_PORTION_ATTN=0: the kernels it replace
     return !v || atoi(v) != 0;
   }();
   return on;
+}
+
+bool latent_tokens_ok(const float* qa, const void* cache, const void* out, int R, int P, int block_size) {
+  return portion_attn_on() && (R == 128 || R == 256 || R == 384 || R == 512) && P >= 0 && P <= 64 && P % 16 == 0 &&
+         shift_of(block_size) >= 0 &&
+         ((reinterpret_cast<uintptr_t>(qa) | reinterpret_cast<uintptr_t>(cache)) & 15) == 0 &&
+         (reinterpret_cast<uintptr_t>(out) & 3) == 0;
+}
+
+int latent_tokens(const float* qa, const void* cache, const int32_t* block_table, int bt_stride, const int32_t* row_seq,
+                  const int32_t* positions, int T, int heads, int R, int P, int block_size, int window, float scale,
+                  const float* sink, const void* gate, int ld_gate, void* out, cudaStream_t st) {
+  int* failed = nullptr;
+  if (!wait_flag(&failed)) {
+    set_error("latent_attn: no mapped host memory");
+    return B200Q_ECUDA;
+  }
+  const LatentTokens a{qa, (const bf16*)cache, block_table, row_seq, positions, sink, (const bf16*)gate, (bf16*)out, failed,
+                       (float)(scale * 1.4426950408889634), bt_stride, heads, R, R + P, shift_of(block_size), window, ld_gate};
+#define BY_RANK(MT)                                             \
+  do {                                                          \
+    if (R == 128) return launch_latent_tokens<MT, 2>(a, T, st); \
+    if (R == 256) return launch_latent_tokens<MT, 4>(a, T, st); \
+    if (R == 384) return launch_latent_tokens<MT, 6>(a, T, st); \
+    return launch_latent_tokens<MT, 8>(a, T, st);               \
+  } while (0)
+  if (heads > 16) BY_RANK(2);
+  BY_RANK(1);
+#undef BY_RANK
 }
 
 bool portion_attn_gqa_ok(const float* qs, const void* cache, const void* out, int kv_heads, int dim, int vdim, int block_size) {
