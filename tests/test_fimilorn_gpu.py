@@ -172,7 +172,7 @@ def standout(T, H, G, D, V, marks, seed):
 
 
 ATTENTION_CASES = [
-    # (T, H, G, D, V, window, marked keys)
+    # (T, H, G, D, V, window, marked keys[, first keys that stay visible behind the window])
     (150, 4, 2, 24, 40, 0, [0, 15, 16, 63, 64, 100]),              # sizes no tile takes
     (200, 2, 1, 64, 64, 64, [0, 15, 16, 63, 64, 127, 128, 135]),   # a window of one tile, pages at its edges
     (300, 4, 4, 128, 128, 0, [7]),                                 # every earlier key: one far back among hundreds
@@ -180,13 +180,16 @@ ATTENTION_CASES = [
     (260, 3, 3, 16, 8, 21, [0, 20, 21, 47, 63, 64, 100, 200]),
     (90, 16, 1, 64, 128, 17, [0, 16, 17, 33, 50]),                 # sixteen heads on one key head
     (70, 24, 1, 128, 64, 0, [0, 18, 40]),                          # more heads per key head than a decode tile has rows
+    (200, 4, 2, 64, 64, 33, [0, 2, 3, 40, 100], 3),                # kept first keys beside a sink
+    (150, 2, 1, 128, 64, 20, [4, 5, 70], 5),
 ]
 
 
-def _attention_want(qs, keys, vals, window, sink, gate):
+def _attention_want(qs, keys, vals, window, sink, gate, kept=0):
     T, H, D = qs.shape
     G, V = keys.shape[1], vals.shape[2]
-    out = O.sink_attention(qs.double(), keys.double(), vals.double(), O.visible(T, window), 1.0,
+    see = O.visible(T, window) | (O.visible(T) & (torch.arange(T)[None, :] < kept))
+    out = O.sink_attention(qs.double(), keys.double(), vals.double(), see, 1.0,
                            sink.double() if sink is not None else None)
     return out * torch.sigmoid(gate.double()).view(T, H, V) if gate is not None else out
 
@@ -199,7 +202,7 @@ def test_attention_sinks_gates_edges_pages_and_far_keys(cuda, case, dtype, how):
     nothing to as strong as that key, with a gate value per channel: whole, in portions beside another sequence, and
     token by token"""
     L, lib = _ops()
-    T, H, G, D, V, window, marks = ATTENTION_CASES[case]
+    T, H, G, D, V, window, marks, kept = (ATTENTION_CASES[case] + (0,))[:8]
     qs, keys, vals = standout(T, H, G, D, V, marks, seed=case)
     g = torch.Generator().manual_seed(100 + case)
     dt, tdt = (L.DTYPE_F32, torch.float32) if dtype == "f32" else (L.DTYPE_BF16, torch.bfloat16)
@@ -207,8 +210,8 @@ def test_attention_sinks_gates_edges_pages_and_far_keys(cuda, case, dtype, how):
     gate = torch.randn(T, H * V + 6, generator=g).to(tdt).float()
     # head h's sink: -20 (nothing), then up to 24, the score of a marked key
     sink = torch.linspace(-20.0, 24.0, H) if H > 1 else torch.tensor([24.0])
-    want = _attention_want(qs, keys, vals, window, sink, gate[:, :H * V])
-    without = _attention_want(qs, keys, vals, window, None, gate[:, :H * V])
+    want = _attention_want(qs, keys, vals, window, sink, gate[:, :H * V], kept)
+    without = _attention_want(qs, keys, vals, window, None, gate[:, :H * V], kept)
     assert float((want - without).abs().max()) > 1.0             # the sinks bite
     paged = Paged(cuda, torch.cat([keys.reshape(T, -1), vals.reshape(T, -1)], 1),
                   torch.cat([torch.zeros(G * D), torch.ones(G * V)]), tdt, case)
@@ -223,7 +226,7 @@ def test_attention_sinks_gates_edges_pages_and_far_keys(cuda, case, dtype, how):
         o = torch.zeros(c + n, H * V, dtype=tdt, device=cuda)
         L.check(lib.b200q_window_attn_sink(q.data_ptr(), paged.cache.data_ptr(), table.data_ptr(), paged.nb,
                                            row_seq.data_ptr(), pos.data_ptr(), desc.data_ptr(), 1 + c, c + n, H, G, D, V,
-                                           paged.bs, window, 0, 0.0, sd.data_ptr(), gs.data_ptr(), H * V + 6, 1, n,
+                                           paged.bs, window, kept, 0.0, sd.data_ptr(), gs.data_ptr(), H * V + 6, 1, n,
                                            o.data_ptr(), dt, None))
         torch.cuda.synchronize()
         if c:   # one key of zeros against the sink: 1 / (1 + exp(sink)), half of it behind the gate
@@ -233,7 +236,7 @@ def test_attention_sinks_gates_edges_pages_and_far_keys(cuda, case, dtype, how):
     tol = 2e-4 if dtype == "f32" else 2e-2
     assert float((got.double().view(T, H, V) - want).abs().max()) < tol * T
     for i in range(T) if H > 1 else []:                         # the marks do what they are meant to (head 0: no sink)
-        seen = [m for m in marks if m <= i and (not window or i - m < window)]
+        seen = [m for m in marks if m <= i and (not window or i - m < window or m < kept)]
         if seen:
             assert abs(float(want[i, 0, 0] / torch.sigmoid(gate[i, 0].double())) - sum(seen) / len(seen)) < 0.5
 
@@ -246,6 +249,8 @@ LATENT_CASES = [
     (256, 2, 128, 16, 0, [5]),                                  # every earlier key: one far back among hundreds
     (120, 20, 256, 64, 33, [0, 32, 33, 64, 65, 97]),            # more heads than one tile has rows
     (300, 16, 512, 64, 129, [0, 127, 128, 129, 255, 256]),
+    (200, 6, 192, 32, 70, [0, 69, 70, 71, 139, 140]),           # tiles, but no whole eighths of the latent
+    (150, 33, 384, 48, 0, [9]),
 ]
 
 
